@@ -56,6 +56,52 @@ class GemvOp(C.Structure):
                 ("h", c_void_p), ("h_amax", c_void_p)]
 
 
+class FLinear(C.Structure):
+    """det_flinear (include/det_b200.h, Part 3)."""
+    _fields_ = [("w", c_void_p), ("N", c_int), ("K", c_int), ("ld", c_int)]
+
+
+class SeqSlot(C.Structure):
+    _fields_ = [("s", c_void_p), ("prev", c_void_p), ("cache", c_void_p)]
+
+
+class SeqRef(C.Structure):
+    _fields_ = [("table", c_void_p), ("one", SeqSlot), ("pos", c_void_p), ("pos0", c_int)]
+
+
+class FNormOp(C.Structure):
+    _fields_ = [("x", c_void_p), ("rows", c_void_p), ("w", c_void_p), ("eps", c_float), ("M", c_int), ("n", c_int),
+                ("dtype", c_int), ("out", c_void_p), ("ld", c_int), ("group_stride", C.c_longlong), ("nmix", c_int),
+                ("mu", c_void_p), ("seq", SeqRef)]
+
+
+class FGemmOp(C.Structure):
+    _fields_ = [("lin", C.POINTER(FLinear)), ("dtype", c_int), ("x", c_void_p), ("ldx", c_int),
+                ("group_stride", C.c_longlong), ("nseg", c_int), ("seg_end", c_int * 8), ("seg_in", c_int * 8),
+                ("glu_from", c_int), ("M", c_int), ("norm_x", c_void_p), ("norm_w", c_void_p), ("eps", c_float),
+                ("y", c_void_p), ("ldy", c_int), ("y_bf16", c_int), ("accumulate", c_int), ("softcap", c_float),
+                ("h", c_void_p), ("ldh", c_int)]
+
+
+class FRecurOp(C.Structure):
+    _fields_ = [("heads", c_int), ("dk", c_int), ("dv", c_int), ("rank", c_int), ("M", c_int), ("dtype", c_int),
+                ("y", c_void_p), ("ldy", c_int), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int),
+                ("gate_off", c_int), ("low_off", c_int), ("q_scale", c_float), ("decay", c_int), ("tau", c_float),
+                ("w2", C.POINTER(FLinear)), ("bias", c_void_p), ("u", c_void_p), ("norm", c_void_p), ("eps", c_float),
+                ("out", c_void_p), ("ldo", c_int), ("scratch", c_void_p), ("seq", SeqRef)]
+
+
+class FLatentOp(C.Structure):
+    _fields_ = [(n, c_int) for n in ("heads", "dim", "rot_dim", "rot_dims", "vdim", "q_rank", "kv_rank", "window")] +                [("scale", c_float), ("cap", c_int), ("M", c_int), ("dtype", c_int), ("y", c_void_p), ("ldy", c_int),
+                ("dq_off", c_int), ("dkv_off", c_int), ("gate_off", c_int), ("dq_norm", c_void_p),
+                ("dkv_norm", c_void_p), ("eps", c_float), ("rope_cos", c_void_p), ("rope_sin", c_void_p),
+                ("cq", c_void_p), ("ldcq", c_int), ("q", c_void_p), ("ldq", c_int), ("wkv", C.POINTER(FLinear)),
+                ("sink", c_void_p), ("out", c_void_p), ("ldo", c_int), ("max_pos", c_int), ("scratch", c_void_p),
+                ("seq", SeqRef)]
+
+
+DET_F32, DET_BF16 = 0, 1
+DET_DECAY_SIGMOID, DET_DECAY_EXP = 0, 1
 DET_LAYOUT_STREAM = 0x100
 DET_LAYOUT_INT8 = 0x200
 DET_LAYOUT_PAIRS = 0x400
@@ -137,6 +183,15 @@ CUDA_ABI = {
     "det_quantize_rows": (None, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
     "det_absmax_heads": (None, [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p]),
     "det_embed_table": (None, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]),
+    "det_f_norm": (None, [C.POINTER(FNormOp), c_void_p]),
+    "det_f_gemm": (None, [C.POINTER(FGemmOp), c_void_p]),
+    "det_f_recur": (None, [C.POINTER(FRecurOp), c_void_p]),
+    "det_f_recur_scratch_bytes": (c_size_t, [c_int, c_int, c_int, c_int]),
+    "det_f_latent_ld": (c_int, [c_int, c_int]),
+    "det_f_latent_scratch_bytes": (c_size_t, [c_int] * 10),
+    "det_f_latent_prep": (None, [C.POINTER(FLatentOp), c_void_p]),
+    "det_f_latent_attn": (None, [C.POINTER(FLatentOp), c_void_p]),
+    "det_debug_set_float": (None, [c_int]),
     "det_attn_set_workspace": (None, [c_void_p, c_size_t]),
     "det_debug_set_attn_tc": (None, [c_int, c_int]),
     "det_debug_set_pdl": (None, [c_int]),
@@ -159,6 +214,17 @@ HOST_API = {
     "dh_cuda_debug": (None, [c_void_p, C.c_uint, c_int]),
     "dh_cuda_test_prim": (None, [c_int, c_void_p, c_size_t, c_size_t, c_size_t, c_void_p, c_size_t]),
     "dh_model_new_synth": (c_void_p, [c_void_p, c_char_p, c_size_t, c_u64, c_size_t, c_size_t]),
+    "dh_model_open": (c_void_p, [c_void_p, c_char_p, c_int, c_size_t, c_size_t]),
+    "dh_hybrid_new_synth": (c_void_p, [c_void_p, c_char_p, c_u64, c_int, c_size_t, c_size_t]),
+    "dh_hybrid_weight_bytes": (c_size_t, [c_void_p]),
+    "dh_hybrid_check_config": (c_int, [c_char_p, C.POINTER(c_size_t)]),
+    "dh_architectures": (c_int, [c_char_p, c_size_t]),
+    "dh_model_forward_rows": (c_int, [c_void_p, c_void_p, c_size_t, c_void_p, c_size_t]),
+    "dh_model_max_batch": (c_size_t, [c_void_p]),
+    "dh_seq_new": (c_void_p, [c_void_p, c_size_t]),
+    "dh_seq_swap": (c_int, [c_void_p, c_void_p]),
+    "dh_seq_clear": (c_int, [c_void_p, c_void_p]),
+    "dh_seq_free": (None, [c_void_p]),
     "dh_model_load": (c_void_p, [c_void_p, c_char_p, c_size_t, c_size_t]),
     "dh_model_calibrated": (c_int, [c_void_p]),
     "dh_write_synthetic_gguf": (c_int, [c_char_p, c_size_t, c_u64, c_char_p, c_size_t]),

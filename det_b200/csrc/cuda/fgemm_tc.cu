@@ -1,0 +1,313 @@
+// Prefill and batched-decode products of the floating-point op set on the 5th-generation tensor cores:
+// tcgen05.mma kind::f16 (bfloat16 x bfloat16 -> fp32) with TMA-fed operands and TMEM accumulators.
+//
+// CTA tile: 128 weight rows (UMMA M, one TMEM lane per row) x TOK tokens (UMMA N: 32, 128 or 256); a stage holds 64 values
+// of K of both operands (128-byte rows, SWIZZLE_128B).  Persistent: a CTA walks its tiles, tokens fastest, with two TMEM
+// accumulators, so that the epilogue of one tile runs beside the loads and products of the next.  Warp 0 issues TMA, warp 1
+// the MMAs, the others drain TMEM and apply the epilogue (residual add, softcap, SwiGLU of interleaved gate / up rows).
+// A launch with few tiles splits K over several CTAs: partial sums go to the library's workspace and the CTA that arrives
+// last adds them in split order, so the result does not depend on the order of arrival.
+#include "umma.cuh"
+#include "fops.cuh"
+#include <algorithm>
+
+namespace detb {
+
+constexpr int FT_ROWS = 128, FT_KE = 64;              // weight rows of a tile, elements of K per stage
+constexpr int FT_A_BYTES = FT_ROWS * 128;
+
+template <int TOK>
+struct FtCfg {
+    static constexpr int B_BYTES = TOK * 128;
+    static constexpr int STAGE_BYTES = FT_A_BYTES + B_BYTES;
+    static constexpr int STAGES = TOK == 256 ? 4 : (TOK == 128 ? 6 : 9);
+    static constexpr int EPI_WARPS = TOK == 32 ? 4 : 8;
+    static constexpr int THREADS = (2 + EPI_WARPS) * 32;
+    static constexpr int EC = TOK * 4 / EPI_WARPS;     // token columns of an epilogue warp
+    static constexpr int TMEM_COLS = 2 * TOK;
+    static constexpr unsigned IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((unsigned)(TOK >> 3) << 17) | ((FT_ROWS >> 4) << 24);
+    static constexpr size_t SMEM = 1024 + (size_t)STAGES * STAGE_BYTES + (2 * STAGES + 4) * 8 + 16;
+};
+
+struct FtPlan {
+    int tok_tiles, items, ksplit, kb;     // kb: stages over the whole of K
+    int m_rows;                           // rows of one input group in the tensor map
+    float* part;
+    unsigned* counters;
+};
+
+__device__ __forceinline__ void umma_bf16(unsigned tmem_d, unsigned long long da, unsigned long long db, unsigned idesc,
+                                          unsigned accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+        ::"r"(tmem_d), "l"(da), "l"(db), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+
+struct FtItem {
+    TilePlace pl;
+    int wt, tt, ks, b0, nb;               // weight tile, token tile, split, first stage and number of stages
+};
+__device__ __forceinline__ FtItem ft_item(const FgemmArgs& a, const FtPlan& p, int i) {
+    FtItem it;
+    it.ks = i % p.ksplit;
+    const int tile = i / p.ksplit;
+    it.tt = tile % p.tok_tiles;
+    it.wt = tile / p.tok_tiles;
+    it.pl = place_tile<FT_ROWS>(a, it.wt);
+    const int per = (p.kb + p.ksplit - 1) / p.ksplit;
+    it.b0 = it.ks * per;
+    it.nb = max(0, min(p.kb, it.b0 + per) - it.b0);
+    return it;
+}
+
+// Two neighbouring tokens (columns) of one weight row: v0 at token m, v1 at token m + 1.
+__device__ __forceinline__ void ft_emit2(const FgemmArgs& a, const TilePlace& pl, int n, int m, float v0, float v1) {
+    if (pl.n0 >= a.glu_from) {
+        // lanes 2i / 2i + 1 hold gate / up: the even lane takes token m, the odd one token m + 1
+        const bool odd = threadIdx.x & 1;
+        const float got = __shfl_xor_sync(FULL, odd ? v0 : v1, 1);
+        const float g = odd ? got : v0, u = odd ? v1 : got;
+        const int mm = m + (odd ? 1 : 0);
+        if (n < pl.n_end && mm < a.M)
+            put(static_cast<bf16*>(a.h) + (size_t)mm * a.ldh + (n - a.glu_from) / 2, silu_fast(g) * u);
+        return;
+    }
+    if (n >= pl.n_end) return;
+    if (a.softcap > 0.0f) {
+        v0 = a.softcap * tanhf(v0 / a.softcap);
+        v1 = a.softcap * tanhf(v1 / a.softcap);
+    }
+    const size_t at = (size_t)m * a.ldy + n;
+    if (a.yb) {
+        if (m < a.M) put(a.yb + at, v0);
+        if (m + 1 < a.M) put(a.yb + at + a.ldy, v1);
+    } else if (a.accumulate) {
+        if (m < a.M) a.y[at] += v0;
+        if (m + 1 < a.M) a.y[at + a.ldy] += v1;
+    } else {
+        if (m < a.M) a.y[at] = v0;
+        if (m + 1 < a.M) a.y[at + a.ldy] = v1;
+    }
+}
+
+template <int TOK>
+__global__ void __launch_bounds__(FtCfg<TOK>::THREADS, 1)
+k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, const FgemmArgs a, const FtPlan p) {
+    using Cfg = FtCfg<TOK>;
+    constexpr int STAGES = Cfg::STAGES;
+    extern __shared__ __align__(1024) uint8_t ft_raw[];
+    uint8_t* stages = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ft_raw) + 1023) & ~(uintptr_t)1023);
+    unsigned long long* full = reinterpret_cast<unsigned long long*>(stages + (size_t)STAGES * Cfg::STAGE_BYTES);
+    unsigned long long* empty = full + STAGES;
+    unsigned long long* tfull = empty + STAGES;      // [2] accumulator complete
+    unsigned long long* tempty = tfull + 2;          // [2] accumulator drained
+    unsigned* tmem_slot = reinterpret_cast<unsigned*>(tempty + 2);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const long long wl = wait_limit(a.error_flag);
+    pdl_trigger();
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < STAGES; s++) {
+            mbar_init(&full[s], 1);
+            mbar_init(&empty[s], 1);
+        }
+        for (int b = 0; b < 2; b++) {
+            mbar_init(&tfull[b], 1);
+            mbar_init(&tempty[b], Cfg::EPI_WARPS);
+        }
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) tmem_alloc(tmem_slot, Cfg::TMEM_COLS);
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const unsigned tmem = *tmem_slot;
+    bool ok = true;
+
+    if (warp == 0) {
+        if (lane == 0) {
+            // the weight boxes of the first stages do not depend on the previous kernel
+            const FtItem first = ft_item(a, p, blockIdx.x);
+            const int lead = min(first.nb, STAGES);
+            for (int l = 0; l < lead; l++) {
+                mbar_expect_tx(&full[l], Cfg::STAGE_BYTES);
+                tma_load_2d(stages + (size_t)l * Cfg::STAGE_BYTES, &map_w, (first.b0 + l) * FT_KE, first.pl.n0, &full[l]);
+            }
+            pdl_wait();
+            unsigned c = 0;                          // stages issued so far
+            for (int i = blockIdx.x; i < p.items && ok; i += gridDim.x) {
+                const FtItem it = ft_item(a, p, i);
+                const int row = a.seg_in[it.pl.seg] * p.m_rows + it.tt * TOK;
+                for (int l = 0; l < it.nb; l++, c++) {
+                    const int s = c % STAGES;
+                    uint8_t* st = stages + (size_t)s * Cfg::STAGE_BYTES;
+                    if (c >= (unsigned)lead) {
+                        ok = mbar_wait(&empty[s], ((c / STAGES) & 1u) ^ 1u, wl);
+                        if (!ok) break;
+                        mbar_expect_tx(&full[s], Cfg::STAGE_BYTES);
+                        tma_load_2d(st, &map_w, (it.b0 + l) * FT_KE, it.pl.n0, &full[s]);
+                    }
+                    tma_load_2d(st + FT_A_BYTES, &map_x, (it.b0 + l) * FT_KE, row, &full[s]);
+                }
+            }
+            if (!ok) {
+                atomicExch(a.error_flag, DETB_ERR_WAIT_EXPIRED);
+                for (unsigned k = 1; k <= (unsigned)STAGES && k <= c; k++)
+                    (void)mbar_wait(&full[(c - k) % STAGES], ((c - k) / STAGES) & 1u, wl);
+            }
+        }
+    } else if (warp == 1) {
+        if (lane == 0) {
+            unsigned c = 0, t = 0;
+            for (int i = blockIdx.x; i < p.items && ok; i += gridDim.x, t++) {
+                const FtItem it = ft_item(a, p, i);
+                const unsigned b = t & 1u;
+                ok = mbar_wait(&tempty[b], ((t >> 1) & 1u) ^ 1u, wl);
+                if (!ok) break;
+                tc_fence_after();
+                for (int l = 0; l < it.nb; l++, c++) {
+                    const int s = c % STAGES;
+                    ok = mbar_wait(&full[s], (c / STAGES) & 1u, wl);
+                    if (!ok) break;
+                    tc_fence_after();
+                    const uint8_t* st = stages + (size_t)s * Cfg::STAGE_BYTES;
+                    const unsigned long long da = umma_desc(st), db = umma_desc(st + FT_A_BYTES);
+#pragma unroll
+                    for (int k = 0; k < 4; k++) umma_bf16(tmem + b * TOK, da + 2 * k, db + 2 * k, Cfg::IDESC, (l | k) ? 1u : 0u);
+                    umma_commit(&empty[s]);
+                }
+                if (ok) umma_commit(&tfull[b]);
+            }
+            if (!ok) atomicExch(a.error_flag, DETB_ERR_WAIT_EXPIRED);
+        }
+    } else {
+        const int q = warp & 3, col0 = ((warp - 2) >> 2) * Cfg::EC, et = threadIdx.x - 64;
+        pdl_wait();
+        unsigned t = 0;
+        for (int i = blockIdx.x; i < p.items && ok; i += gridDim.x, t++) {
+            const FtItem it = ft_item(a, p, i);
+            const unsigned b = t & 1u;
+            ok = mbar_wait(&tfull[b], (t >> 1) & 1u, wl);
+            if (!ok) break;
+            tc_fence_after();
+            const int n = it.pl.n0 + q * 32 + lane, m0 = it.tt * TOK + col0;
+            const unsigned taddr = tmem + ((unsigned)(q * 32) << 16) + b * TOK + col0;
+            if (p.ksplit == 1) {
+                for (int c = 0; c < Cfg::EC; c += 32) {
+                    int r[32];
+                    tmem_ld(taddr + c, r);
+                    tmem_wait_ld();
+                    if (c + 32 >= Cfg::EC) {
+                        tc_fence_before();
+                        __syncwarp();
+                        if (lane == 0) mbar_arrive(&tempty[b]);
+                    }
+                    if (m0 + c < a.M) {
+#pragma unroll
+                        for (int j = 0; j < 32; j += 2)
+                            ft_emit2(a, it.pl, n, m0 + c + j, __int_as_float(r[j]), __int_as_float(r[j + 1]));
+                    }
+                }
+            } else {
+                // split K (TOK == 32, four epilogue warps, EC == 32): one partial tile per split
+                __shared__ unsigned last_cta;
+                const int tile = i / p.ksplit;
+                int r[32];
+                tmem_ld(taddr, r);
+                tmem_wait_ld();
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&tempty[b]);
+                float* mine = p.part + ((size_t)tile * p.ksplit + it.ks) * (FT_ROWS * 32) + q * 32 + lane;
+#pragma unroll
+                for (int j = 0; j < 32; j++) mine[j * FT_ROWS] = __int_as_float(r[j]);
+                __threadfence();
+                asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
+                if (et == 0) last_cta = atomicAdd(p.counters + tile, 1u) == (unsigned)p.ksplit - 1;
+                asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
+                if (last_cta) {
+                    __threadfence();
+                    const float* all = p.part + (size_t)tile * p.ksplit * (FT_ROWS * 32) + q * 32 + lane;
+                    float v[32];
+#pragma unroll
+                    for (int j = 0; j < 32; j++) v[j] = 0.0f;
+                    for (int s = 0; s < p.ksplit; s++)
+#pragma unroll
+                        for (int j = 0; j < 32; j++)
+                            if (m0 + j < a.M) v[j] += __ldcg(all + (size_t)s * (FT_ROWS * 32) + j * FT_ROWS);
+                    if (et == 0) p.counters[tile] = 0;
+#pragma unroll
+                    for (int j = 0; j < 32; j += 2)
+                        if (m0 + j < a.M) ft_emit2(a, it.pl, n, m0 + j, v[j], v[j + 1]);
+                }
+                asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");   // last_cta is read before it is written again
+            }
+        }
+        if (!ok && lane == 0) atomicExch(a.error_flag, DETB_ERR_WAIT_EXPIRED);
+    }
+    tc_fence_before();
+    __syncthreads();
+    if (warp == 1) tmem_dealloc(tmem, Cfg::TMEM_COLS);
+}
+
+// A [rows][ld] bfloat16 matrix as a map with 64-column boxes (128 bytes, swizzled), zero fill outside.
+static CUtensorMap bf16_map(const void* base, size_t rows, int ld, int box_rows) {
+    CUtensorMap map;
+    const cuuint64_t dims[2] = {(cuuint64_t)ld, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)FT_KE, (cuuint32_t)box_rows};
+    const cuuint32_t estr[2] = {1, 1};
+    const CUresult r = encode_fn()(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+                                   CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                                   CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    DETB_REQUIRE(r == CUDA_SUCCESS, "cuTensorMapEncodeTiled failed");
+    return map;
+}
+
+template <int TOK>
+static void launch_tok(FgemmArgs a, cudaStream_t q) {
+    using Cfg = FtCfg<TOK>;
+    plan_tiles(a, FT_ROWS);
+    int groups = 1;
+    for (int s = 0; s < a.nseg; s++) groups = std::max(groups, a.seg_in[s] + 1);
+    FtPlan p{};
+    p.tok_tiles = (a.M + TOK - 1) / TOK;
+    p.kb = (a.K + FT_KE - 1) / FT_KE;
+    p.ksplit = 1;
+    const int tiles = a.tile0[a.nseg] * p.tok_tiles, sms = sm_count();
+    if (TOK == 32 && !(float_flags() & 4)) {
+        size_t bytes = 0;
+        int ncnt = 0;
+        p.part = fsplit_workspace(&bytes);
+        p.counters = fsplit_counters(&ncnt);
+        // fill the SMs, at least four stages of K per CTA
+        const int want = std::min({sms / std::max(tiles, 1), p.kb / 4, 16});
+        if (want > 1 && tiles <= ncnt && (size_t)tiles * want * FT_ROWS * 32 * sizeof(float) <= bytes) p.ksplit = want;
+        // every split owns at least one stage
+        while (p.ksplit > 1 && (p.ksplit - 1) * ((p.kb + p.ksplit - 1) / p.ksplit) >= p.kb) p.ksplit--;
+    }
+    p.items = tiles * p.ksplit;
+    // input groups lie gstride elements apart; a map row is one row of the buffer
+    DETB_REQUIRE(groups == 1 || a.gstride % a.ldx == 0, "input groups must be whole rows apart");
+    p.m_rows = groups == 1 ? 0 : (int)(a.gstride / a.ldx);
+    const size_t x_rows = (size_t)(groups - 1) * p.m_rows + a.M;
+    DETB_REQUIRE(a.ldw == round8(a.K), "linear: weight rows must be padded to 8 elements");
+    const CUtensorMap map_w = bf16_map(a.w, a.N, a.ldw, FT_ROWS);
+    const CUtensorMap map_x = bf16_map(a.x, x_rows, a.ldx, TOK);
+    static bool configured = false;
+    if (!configured) {
+        DETB_CUDA_OK(cudaFuncSetAttribute(k_fgemm_tc<TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM));
+        configured = true;
+    }
+    launch_pdl(k_fgemm_tc<TOK>, dim3(std::min(p.items, sms)), dim3(Cfg::THREADS), Cfg::SMEM, q, 1, map_w, map_x, a, p);
+}
+
+void fgemm_tc_launch(FgemmArgs a, cudaStream_t q) {
+    if (a.M <= 32) launch_tok<32>(a, q);
+    else if (a.M <= 128) launch_tok<128>(a, q);
+    else launch_tok<256>(a, q);
+}
+
+}  // namespace detb

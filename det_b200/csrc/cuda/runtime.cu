@@ -25,10 +25,14 @@ struct Runtime {
     // scratch owned by the library, allocated once here so that no call path ever allocates:
     unsigned long long* splitk_cells = nullptr;   // split-K partial sums of the tensor-core GEMM, zero between calls
     unsigned* splitk_counters = nullptr;
+    float* fsplit_ws = nullptr;                   // split-K partial sums of the floating-point GEMM, and its counters
+    unsigned* fsplit_counters = nullptr;
     void* attn_ws = nullptr;                      // workspace of the tensor-core prefill attention
     size_t attn_ws_bytes = 0;
     bool attn_ws_owned = false;
 };
+constexpr size_t FSPLIT_BYTES = 8u << 20;
+constexpr int FSPLIT_TILES = 512;
 Runtime* g_rt = nullptr;
 std::once_flag g_once;
 
@@ -61,6 +65,8 @@ void bring_up() {
     if (cudaMalloc(&rt->splitk_cells, ncell * 8) != cudaSuccess || cudaMemset(rt->splitk_cells, 0, ncell * 8) != cudaSuccess ||
         cudaMalloc(&rt->splitk_counters, 4 * tiles * sizeof(unsigned)) != cudaSuccess ||      // tiles as narrow as 32 tokens
         cudaMemset(rt->splitk_counters, 0, 4 * tiles * sizeof(unsigned)) != cudaSuccess) { delete rt; return; }
+    if (cudaMalloc(&rt->fsplit_ws, FSPLIT_BYTES) != cudaSuccess || cudaMalloc(&rt->fsplit_counters, FSPLIT_TILES * sizeof(unsigned)) != cudaSuccess ||
+        cudaMemset(rt->fsplit_counters, 0, FSPLIT_TILES * sizeof(unsigned)) != cudaSuccess) { delete rt; return; }
     // DET_B200_ATTN_WS_MB sizes the attention workspace (default 256; 0: none, prefill attention then stays on the CUDA cores
     // until det_attn_set_workspace provides one)
     size_t ws_mb = 256;
@@ -96,6 +102,14 @@ size_t smem_optin() { return rt().smem_optin; }
 int* error_word() { return rt().error_word; }
 unsigned long long* splitk_cells() { return rt().splitk_cells; }
 unsigned* splitk_counters() { return rt().splitk_counters; }
+float* fsplit_workspace(size_t* bytes) {
+    *bytes = FSPLIT_BYTES;
+    return rt().fsplit_ws;
+}
+unsigned* fsplit_counters(int* n) {
+    *n = FSPLIT_TILES;
+    return rt().fsplit_counters;
+}
 void* attn_workspace(size_t* bytes) {
     *bytes = rt().attn_ws_bytes;
     return rt().attn_ws;

@@ -25,6 +25,8 @@ __device__ __forceinline__ long long wait_limit(const int* error_flag) {
 unsigned long long* splitk_cells();
 unsigned* splitk_counters();
 void* attn_workspace(size_t* bytes);
+float* fsplit_workspace(size_t* bytes);   // split-K partial sums of the floating-point GEMM
+unsigned* fsplit_counters(int* n);        // ... and its tile counters, zero between calls
 
 bool pdl_enabled();
 

@@ -3,11 +3,13 @@
 // GdnShape, trait Backend).  Names, argument order and meaning follow the trait so that the driver
 // (model.hpp, the mirror of qwen35.rs / model.rs) and the conformance suites read like the reference's.
 #pragma once
+#include "det_b200.h"
 #include <cmath>
 #include <cstddef>
 #include <cstdint>
 #include <cstring>
 #include <memory>
+#include <stdexcept>
 #include <string>
 #include <utility>
 #include <vector>
@@ -125,12 +127,30 @@ struct GdnShape {
     float eps;
 };
 
+// ---- floating-point op set (models whose linears stay in bfloat16; not in the reference trait)
+enum class Dtype { F32 = DET_F32, BF16 = DET_BF16 };   // the activations that enter a linear
+inline size_t dtype_bytes(Dtype d) { return d == Dtype::BF16 ? 2 : 4; }
+// W[n][ld] bfloat16 in backend memory, ld = k rounded up to 8, zeros behind column k.
+struct FLinear {
+    Buf<uint16_t> w;
+    size_t n = 0, k = 0, ld = 0;
+    det_flinear view() const { return det_flinear{w.ptr(), (int)n, (int)k, (int)ld}; }
+};
+// What one sequence keeps in one layer; a layer uses the members it needs.
+struct FloatState {
+    Buf<float> s;          // recurrent state [heads][dk][dv]
+    Buf<float> prev;       // the previous token's normalised row
+    Buf<uint8_t> cache;    // `cap` cache rows, used as a ring
+    size_t cap = 0;
+};
+
 // The per-sequence caches (attention layer) or states (GDN layer) behind the rows of a batched decode step: row b of
 // the step's activations is the current token of sequence b.  A backend may attach its own lookup tables.
 struct RowSet {
     virtual ~RowSet() = default;
     std::vector<const KvCache*> kv;
     std::vector<const GdnState*> st;
+    std::vector<const FloatState*> fs;
 };
 
 // backend.rs:203-302
@@ -217,6 +237,19 @@ class Backend {
         for (size_t r = 0; r < rows; r++) out[r] = sample(Buf<float>::view(logits.ptr_at(r * v), v), v, inv_temp, top_k, top_p, z[r]);
         return out;
     }
+    // ---- floating-point op set; the operation structs and their meaning are those of include/det_b200.h, Part 3.  A backend
+    // that carries quantized models only keeps these defaults.
+    virtual void synth_bf16(uint64_t, uint64_t, size_t, uint16_t*) { no_float_ops(); }   // elements of a seeded tensor
+    // x[i] = row ids[i] of a table of ggml type `type`; ids in backend memory
+    virtual void embed(const void*, int, const Buf<int32_t>&, size_t, size_t, const Buf<float>&) { no_float_ops(); }
+    virtual std::unique_ptr<RowSet> make_slots(std::vector<const FloatState*>) { no_float_ops(); return nullptr; }
+    // The sequence reference of a step: `t` tokens of `st` from pos0 on, or one row per sequence of `rows`.
+    virtual det_seq_ref seq_ref(const FloatState&, size_t, const RowSet*, const Buf<int32_t>*) { no_float_ops(); return {}; }
+    virtual void f_norm(const det_fnorm_op&) { no_float_ops(); }
+    virtual void f_gemm(const det_fgemm_op&) { no_float_ops(); }
+    virtual void f_recur(const det_frecur_op&) { no_float_ops(); }             // the backend supplies `scratch`
+    virtual void f_latent_prep(const det_flatent_op&) { no_float_ops(); }
+    virtual void f_latent_attn(const det_flatent_op&, size_t) { no_float_ops(); }   // supplies `scratch`; bound on any position
     virtual int32_t argmax(const Buf<float>& logits, size_t v) = 0;
     virtual int32_t sample(const Buf<float>& logits, size_t v, float inv_temp, size_t top_k, float top_p,
                            uint64_t z) = 0;
@@ -250,6 +283,9 @@ class Backend {
     }
     template <class T>
     void zero(const Buf<T>& b) { zero_bytes(b.ptr(), b.bytes()); }
+
+  private:
+    [[noreturn]] static void no_float_ops() { throw std::runtime_error("this backend has no floating-point op set"); }
 };
 
 inline void Backend::attention_rows(const AttnLayer& l, const RowSet& rows, const Buf<int32_t>& pos, size_t,

@@ -3,7 +3,9 @@
 #include "convert.hpp"
 #include "cuda_backend.hpp"
 #include "graph_decode.hpp"
-#include "model.hpp"
+#include "hybrid.hpp"
+#include "qwen35.hpp"
+#include "registry.hpp"
 #include "serve.hpp"
 #include <cstring>
 #include <functional>
@@ -24,6 +26,17 @@ int guarded(F&& f) {
         return fail(ex.what());
     }
 }
+// The quantized model behind a handle; throws when it is of another class.
+det::Qwen35Model& qwen(void* m) {
+    auto* q = dynamic_cast<det::Qwen35Model*>(static_cast<det::Model*>(m));
+    if (!q) throw std::runtime_error("this call needs a qwen35 model");
+    return *q;
+}
+// A sequence held beside a model: its caches and position while another one is bound.
+struct HeldSequence {
+    std::unique_ptr<det::SeqCache> cache;
+    size_t pos = 0;
+};
 }  // namespace
 
 extern "C" {
@@ -71,17 +84,96 @@ void* dh_model_new_synth(void* backend, const char* config, size_t layers, uint6
                          size_t max_batch) {
     try {
         det::Config cfg = det::config_by_name(config, layers);
-        return det::Model::load_synthetic(cfg, seed, static_cast<det::Backend*>(backend), max_ctx, max_batch).release();
+        return static_cast<det::Model*>(det::Qwen35Model::load_synthetic(cfg, seed, static_cast<det::Backend*>(backend), max_ctx, max_batch).release());
     } catch (const std::exception& ex) {
         g_err = ex.what();
         return nullptr;
     }
 }
+// ---- any checkpoint, its class found through the registry: a folder (config.json + model.safetensors) or a det GGUF.  dtype:
+// DET_BF16 or DET_F32, the activations of a floating-point model.
+void* dh_model_open(void* backend, const char* path, int dtype, size_t max_ctx, size_t max_batch) {
+    try {
+        det::OpenOptions o;
+        o.max_ctx = max_ctx;
+        o.max_batch = max_batch;
+        o.dtype = dtype == DET_F32 ? det::Dtype::F32 : det::Dtype::BF16;
+        return det::open_model(path, static_cast<det::Backend*>(backend), o).release();
+    } catch (const std::exception& ex) {
+        g_err = ex.what();
+        return nullptr;
+    }
+}
+// A hybrid model of the given configuration (the text of a config.json) with seeded random weights.
+void* dh_hybrid_new_synth(void* backend, const char* config, uint64_t seed, int dtype, size_t max_ctx, size_t max_batch) {
+    try {
+        return static_cast<det::Model*>(det::HybridModel::load_synthetic(det::Json::parse(config), seed, static_cast<det::Backend*>(backend),
+                                                                         max_ctx, max_batch,
+                                                                         dtype == DET_F32 ? det::Dtype::F32 : det::Dtype::BF16).release());
+    } catch (const std::exception& ex) {
+        g_err = ex.what();
+        return nullptr;
+    }
+}
+size_t dh_hybrid_weight_bytes(void* m) {
+    auto* h = dynamic_cast<det::HybridModel*>(static_cast<det::Model*>(m));
+    return h ? h->weight_bytes() : 0;
+}
+// Parses and checks a hybrid configuration without building anything; writes the number of layers.
+int dh_hybrid_check_config(const char* config, size_t* n_layers) {
+    return guarded([&] {
+        *n_layers = det::HybridConfig::from_json(det::Json::parse(config)).layers.size();
+        return std::string();
+    });
+}
+// The registered architecture names, separated by spaces.
+int dh_architectures(char* out, size_t cap) {
+    return guarded([&] {
+        std::string s;
+        for (const det::Architecture& a : det::architectures()) s += (s.empty() ? "" : " ") + std::string(a.name);
+        snprintf(out, cap, "%s", s.c_str());
+        return std::string();
+    });
+}
+// One step with the logits of the given rows (places among ids), in that order, for dh_model_logits.
+int dh_model_forward_rows(void* m, const int32_t* ids, size_t t, const int32_t* want, size_t n_want) {
+    return guarded([&] { return static_cast<det::Model*>(m)->forward_rows(ids, t, std::vector<int32_t>(want, want + n_want)); });
+}
+// ---- further sequences of a model: a handle holds the caches and the position of one that is not bound; swap exchanges it
+// with the bound one
+void* dh_seq_new(void* m, size_t ctx) {
+    try {
+        auto s = std::make_unique<HeldSequence>();
+        s->cache = static_cast<det::Model*>(m)->new_sequence(ctx);
+        return s.release();
+    } catch (const std::exception& ex) {
+        g_err = ex.what();
+        return nullptr;
+    }
+}
+int dh_seq_swap(void* m, void* seq) {
+    return guarded([&] {
+        auto* model = static_cast<det::Model*>(m);
+        auto* s = static_cast<HeldSequence*>(seq);
+        model->swap_sequence(*s->cache);
+        std::swap(model->pos, s->pos);
+        return std::string();
+    });
+}
+int dh_seq_clear(void* m, void* seq) {
+    return guarded([&] {
+        auto* s = static_cast<HeldSequence*>(seq);
+        static_cast<det::Model*>(m)->clear_sequence(*s->cache);
+        s->pos = 0;
+        return std::string();
+    });
+}
+void dh_seq_free(void* seq) { delete static_cast<HeldSequence*>(seq); }
 // ---- det files: Model::load, the synthetic writers, convert, calibrate
 void* dh_model_load(void* backend, const char* path, size_t max_ctx, size_t max_batch) {
     try {
         std::string err;
-        std::unique_ptr<det::Model> m = det::Model::load(path, static_cast<det::Backend*>(backend), max_ctx, max_batch, err);
+        std::unique_ptr<det::Model> m = det::Qwen35Model::load(path, static_cast<det::Backend*>(backend), max_ctx, max_batch, err);
         if (!m) g_err = err;
         return m.release();
     } catch (const std::exception& ex) {
@@ -89,7 +181,7 @@ void* dh_model_load(void* backend, const char* path, size_t max_ctx, size_t max_
         return nullptr;
     }
 }
-int dh_model_calibrated(void* m) { return static_cast<det::Model*>(m)->calibrated ? 1 : 0; }
+int dh_model_calibrated(void* m) { return qwen(m).calibrated ? 1 : 0; }
 int dh_write_synthetic_gguf(const char* config, size_t layers, uint64_t seed, const char* path, size_t n_pos) {
     return guarded([&] { return det::write_synthetic_gguf(det::config_by_name(config, layers), seed, path, n_pos); });
 }
@@ -132,7 +224,7 @@ int dh_convert_default_output(const char* src_path, const char* bits, char* out,
 int dh_v_scales(void* m, const int32_t* ids, size_t n, float* out, size_t cap, size_t* n_out) {
     return guarded([&] {
         std::vector<float> s;
-        std::string e = det::v_scales(*static_cast<det::Model*>(m), ids, n, s);
+        std::string e = det::v_scales(qwen(m), ids, n, s);
         if (!e.empty()) return e;
         *n_out = s.size();
         std::memcpy(out, s.data(), std::min(cap, s.size()) * sizeof(float));
@@ -146,13 +238,13 @@ void dh_calibration_ids(const int32_t* prefix, size_t n_prefix, size_t vocab, si
 // calibrate.rs:91-109.  in_place: 0 on success, 2 when the header has no room (nothing written); copy: 0 on success.
 int dh_write_scales_in_place(void* m, const float* scales, size_t n, const char* path) {
     std::string err;
-    if (det::write_scales_in_place(*static_cast<det::Model*>(m), std::vector<float>(scales, scales + n), path, err)) return 0;
+    if (det::write_scales_in_place(qwen(m), std::vector<float>(scales, scales + n), path, err)) return 0;
     if (err.empty()) return 2;
     return fail(err);
 }
 int dh_write_scales_copy(void* m, const float* scales, size_t n, const char* out) {
     std::string err;
-    return det::write_scales_copy(*static_cast<det::Model*>(m), std::vector<float>(scales, scales + n), out, err) ? 0 : fail(err);
+    return det::write_scales_copy(qwen(m), std::vector<float>(scales, scales + n), out, err) ? 0 : fail(err);
 }
 // ---- container access for tools and tests: a handle is a std::shared_ptr<det::Gguf>*
 void* dh_gguf_open(const char* path) {
@@ -322,15 +414,16 @@ void* dh_model_new_synth_tp(void* backend, const char* config, size_t layers, ui
                             size_t max_batch, void* comm) {
     try {
         det::Config cfg = det::config_by_name(config, layers);
-        return det::Model::load_synthetic(cfg, seed, static_cast<det::Backend*>(backend), max_ctx, max_batch,
-                                          static_cast<det::Comm*>(comm)).release();
+        return static_cast<det::Model*>(det::Qwen35Model::load_synthetic(cfg, seed, static_cast<det::Backend*>(backend), max_ctx,
+                                                                         max_batch, static_cast<det::Comm*>(comm)).release());
     } catch (const std::exception& ex) {
         g_err = ex.what();
         return nullptr;
     }
 }
 void dh_model_free(void* m) { delete static_cast<det::Model*>(m); }
-size_t dh_model_vocab(void* m) { return static_cast<det::Model*>(m)->cfg.vocab; }
+size_t dh_model_vocab(void* m) { return static_cast<det::Model*>(m)->vocab(); }
+size_t dh_model_max_batch(void* m) { return static_cast<det::Model*>(m)->max_batch; }
 size_t dh_model_pos(void* m) { return static_cast<det::Model*>(m)->pos; }
 int dh_model_set_all_logits(void* m, int all) {
     return guarded([&] {
@@ -455,7 +548,7 @@ size_t dh_batch_tokens(void* b, size_t i, int32_t* out, size_t cap) {
 // One decoded token's GEMVs, `reps` times, without syncing in between (the caller times it with events on the queue).
 int dh_gemv_sweep(void* m, int reps, size_t* bytes, size_t* launches) {
     return guarded([&] {
-        det::GemvSweep r = det::gemv_sweep(*static_cast<det::Model*>(m), reps);
+        det::GemvSweep r = det::gemv_sweep(qwen(m), reps);
         *bytes = r.bytes;
         *launches = r.launches;
         return std::string();

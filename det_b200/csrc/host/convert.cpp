@@ -492,7 +492,7 @@ struct AbsMax : Observer {   // calibrate.rs:12-36; the fold itself is the backe
 };
 }  // namespace
 
-std::string v_scales(Model& m, const int32_t* ids, size_t n, std::vector<float>& scales) {
+std::string v_scales(Qwen35Model& m, const int32_t* ids, size_t n, std::vector<float>& scales) {
     AbsMax obs;
     obs.n_kv = m.cfg.n_kv;
     obs.hd = m.cfg.head_dim;
@@ -508,14 +508,14 @@ std::string v_scales(Model& m, const int32_t* ids, size_t n, std::vector<float>&
     return "";
 }
 
-bool write_scales_in_place(const Model& m, const std::vector<float>& scales, const std::string& path, std::string& err) {
+bool write_scales_in_place(const Qwen35Model& m, const std::vector<float>& scales, const std::string& path, std::string& err) {
     if (!m.gguf) {
         err = "the model was not loaded from a file";
         return false;
     }
     return m.gguf->set_metadata_in_place(path, V_SCALE_KEY, GgufValue::f32_array(scales), err);
 }
-bool write_scales_copy(const Model& m, const std::vector<float>& scales, const std::string& out, std::string& err) {
+bool write_scales_copy(const Qwen35Model& m, const std::vector<float>& scales, const std::string& out, std::string& err) {
     if (!m.gguf) {
         err = "the model was not loaded from a file";
         return false;

@@ -6,7 +6,7 @@
 // CUDA backend (cuda_quantize_rows, same bytes).
 #pragma once
 #include "gguf.hpp"
-#include "model.hpp"
+#include "qwen35.hpp"
 #include <functional>
 
 namespace det {
@@ -57,9 +57,9 @@ constexpr float HEADROOM = 8.0f;   // calibrate.rs:10
 // The generator part of calibrate.rs:38-64: `prefix` (the caller's tokenized text, may be empty) followed by n_random ids.
 std::vector<int32_t> calibration_ids(const std::vector<int32_t>& prefix, size_t vocab, size_t n_random);
 // calibrate.rs:66-89 — runs `ids` through the model and returns the per-(attention layer, kv head) value scales.
-std::string v_scales(Model& m, const int32_t* ids, size_t n, std::vector<float>& scales);
+std::string v_scales(Qwen35Model& m, const int32_t* ids, size_t n, std::vector<float>& scales);
 // calibrate.rs:91-109
-bool write_scales_in_place(const Model& m, const std::vector<float>& scales, const std::string& path, std::string& err);
-bool write_scales_copy(const Model& m, const std::vector<float>& scales, const std::string& out, std::string& err);
+bool write_scales_in_place(const Qwen35Model& m, const std::vector<float>& scales, const std::string& path, std::string& err);
+bool write_scales_copy(const Qwen35Model& m, const std::vector<float>& scales, const std::string& out, std::string& err);
 
 }  // namespace det

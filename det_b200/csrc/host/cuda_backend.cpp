@@ -4,7 +4,7 @@
 // picks back through a one-element device buffer.  The B200-specific part is linear(): besides the reference layout
 // (kept for large-M GEMMs) it builds the streaming layout the decode GEMV reads (det_linear_repack).
 #include "cuda_backend.hpp"
-#include "model.hpp"
+#include "qwen35.hpp"
 #include <cstdio>
 #include <cstdlib>
 #include <stdexcept>
@@ -543,6 +543,65 @@ void CudaBackend::silu_mul(const Buf<float>& g, const Buf<float>& u, size_t m, s
     det_silu_mul_quant(g.ptr(), u.ptr(), (int)m, (int)n, h.ptr(), nullptr, nullptr, nullptr, ST);
 }
 
+// ---- floating-point op set
+void CudaBackend::synth_bf16(uint64_t seed, uint64_t tid, size_t count, uint16_t* out) {
+    flush_pending();
+    det_synth_bf16(seed, tid, (long long)count, out, ST);
+}
+void CudaBackend::embed(const void* table, int type, const Buf<int32_t>& ids, size_t t, size_t h, const Buf<float>& x) {
+    flush_pending();
+    det_embed_table(table, type, ids.ptr(), (int)t, (int)h, x.ptr(), ST);
+}
+std::unique_ptr<RowSet> CudaBackend::make_slots(std::vector<const FloatState*> fs) {
+    auto r = std::make_unique<CudaRowSet>();
+    std::vector<det_seq_slot> t;
+    for (const FloatState* f : fs) t.push_back(det_seq_slot{f->s.ptr(), f->prev.ptr(), f->cache.ptr()});
+    r->table = upload(reinterpret_cast<const uint8_t*>(t.data()), t.size() * sizeof(det_seq_slot));
+    sync();   // the staging vector dies here
+    r->fs = std::move(fs);
+    return r;
+}
+det_seq_ref CudaBackend::seq_ref(const FloatState& st, size_t pos0, const RowSet* rows, const Buf<int32_t>* pos) {
+    det_seq_ref r{};
+    if (rows) {
+        const CudaRowSet* rs = dynamic_cast<const CudaRowSet*>(rows);
+        if (!rs || !pos) throw std::logic_error("the row set belongs to another backend");
+        r.table = reinterpret_cast<const det_seq_slot*>(rs->table.ptr());
+        r.pos = pos->ptr();
+        return r;
+    }
+    r.one = det_seq_slot{st.s.ptr(), st.prev.ptr(), st.cache.ptr()};
+    r.pos = pos_dev;
+    r.pos0 = (int)pos0;
+    return r;
+}
+void CudaBackend::f_norm(const det_fnorm_op& op) {
+    flush_pending();
+    det_f_norm(&op, ST);
+}
+void CudaBackend::f_gemm(const det_fgemm_op& op) {
+    flush_pending();
+    det_f_gemm(&op, ST);
+}
+void CudaBackend::f_recur(const det_frecur_op& op_) {
+    flush_pending();
+    det_frecur_op op = op_;
+    op.scratch = scratch(float_scratch_, det_f_recur_scratch_bytes(op.M, op.heads, op.dk, op.dv));
+    det_f_recur(&op, ST);
+}
+void CudaBackend::f_latent_prep(const det_flatent_op& op) {
+    flush_pending();
+    det_f_latent_prep(&op, ST);
+}
+void CudaBackend::f_latent_attn(const det_flatent_op& op_, size_t max_ctx) {
+    flush_pending();
+    det_flatent_op op = op_;
+    if (pos_dev && !op.seq.table) op.max_pos = max_pos;
+    op.scratch = scratch(float_scratch_, det_f_latent_scratch_bytes(op.M, op.heads, op.dim, op.rot_dim, op.vdim, op.kv_rank, op.window,
+                                                                    op.cap, (int)max_ctx - 1, op.dtype));
+    det_f_latent_attn(&op, ST);
+}
+
 // cuda.rs:425-471
 int32_t CudaBackend::argmax(const Buf<float>& logits, size_t v) {
     flush_pending();
@@ -620,11 +679,11 @@ void CudaBackend::absmax_heads(const Buf<float>& v, size_t t, size_t heads, size
 }
 
 // Every linear of the model once at M = 1 (the launches of one decoded token's GEMVs), `reps` times.
-GemvSweep gemv_sweep(Model& m, int reps) {
+GemvSweep gemv_sweep(Qwen35Model& m, int reps) {
     GemvSweep r{0, 0};
     CudaBackend* bk = dynamic_cast<CudaBackend*>(m.backend);
     if (!bk) throw std::runtime_error("gemv_sweep needs the CUDA backend");
-    const Buf<float>& y = m.w.logits;   // widest output of any linear; nothing is allocated or freed in here
+    const Buf<float>& y = m.logits_buf;   // widest output of any linear; nothing is allocated or freed in here
     auto run = [&](const Proj& p, const Buf<int8_t>& xq, const Buf<float>& sx, const Buf<uint16_t>& mx) {
         for (const auto& lin : p.lins) {
             bk->gemm(*lin, xq, sx, mx, 1, GemmOut::write(y));

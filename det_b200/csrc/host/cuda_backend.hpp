@@ -56,6 +56,15 @@ class CudaBackend : public Backend {
     void absmax_heads(const Buf<float>& v, size_t t, size_t heads, size_t hd, const Buf<float>& slots) override;
     void add(const Buf<float>& x, const Buf<float>& y, size_t n) override;
     void silu_mul(const Buf<float>& g, const Buf<float>& u, size_t m, size_t n, const Buf<float>& h) override;
+    void synth_bf16(uint64_t seed, uint64_t tid, size_t count, uint16_t* out) override;
+    void embed(const void* table, int type, const Buf<int32_t>& ids, size_t t, size_t h, const Buf<float>& x) override;
+    std::unique_ptr<RowSet> make_slots(std::vector<const FloatState*> fs) override;
+    det_seq_ref seq_ref(const FloatState& st, size_t pos0, const RowSet* rows, const Buf<int32_t>* pos) override;
+    void f_norm(const det_fnorm_op& op) override;
+    void f_gemm(const det_fgemm_op& op) override;
+    void f_recur(const det_frecur_op& op) override;
+    void f_latent_prep(const det_flatent_op& op) override;
+    void f_latent_attn(const det_flatent_op& op, size_t max_ctx) override;
     int32_t argmax(const Buf<float>& logits, size_t v) override;
     int32_t sample(const Buf<float>& logits, size_t v, float inv_temp, size_t top_k, float top_p, uint64_t z) override;
 
@@ -133,7 +142,7 @@ class CudaBackend : public Backend {
     void issue_gemm_tc(const PendingGemm& g, const CudaLinear* second, const std::vector<float*>* dsts2);
     void* scratch(Buf<uint8_t>& slot, size_t bytes);
     void finish_linear(CudaLinear& l);
-    Buf<uint8_t> attn_scratch_, gdn_scratch_, sample_scratch_, synth_scratch_;
+    Buf<uint8_t> attn_scratch_, gdn_scratch_, sample_scratch_, synth_scratch_, float_scratch_;
     Buf<float> swiglu_h_;            // SwiGLU product of a fused gate|up GEMV (the next GEMV quantizes it in its prologue)
     Buf<uint32_t> swiglu_amax_;      // its group maxima, folded by that GEMV's epilogue and consumed by the next one's prologue
     Buf<int32_t> pick_, picks_;
@@ -146,13 +155,13 @@ std::vector<uint8_t> cuda_synth_det_rows(uint64_t seed, uint64_t tid, size_t src
 void cuda_quantize_rows(const uint8_t* src, int ggml_type, size_t src_rows, const std::vector<int>* row_perm,
                         const std::vector<int>* col_perm, size_t n, size_t k, int bits, uint8_t* out);
 
-class Model;
+class Qwen35Model;
 struct GemvSweep {
     size_t bytes;      // algorithmic bytes moved: weights + scales + activations in + outputs
     size_t launches;
 };
 // Issues the GEMV of every linear of the model at M = 1 (one decoded token's worth), `reps` times, into the model's
 // logits buffer; no allocation and no sync inside.  The caller brackets it with events to get the GEMV-only rate.
-GemvSweep gemv_sweep(Model& m, int reps);
+GemvSweep gemv_sweep(Qwen35Model& m, int reps);
 
 }  // namespace det

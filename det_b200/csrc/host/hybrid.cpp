@@ -1,0 +1,656 @@
+#include "hybrid.hpp"
+#include "safetensors.hpp"
+#include "synth.hpp"
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+#include <stdexcept>
+
+namespace det {
+
+namespace {
+size_t round8(size_t n) { return (n + 7) & ~(size_t)7; }
+[[noreturn]] void bad(const std::string& what) { throw std::runtime_error(what); }
+}  // namespace
+
+// ---------------------------------------------------------------------------------------------------- configuration
+HybridConfig HybridConfig::from_json(const Json& j) {
+    HybridConfig c;
+    c.vocab = j.size("vocab");
+    c.width = j.size("width");
+    c.eps = (float)j.at("norm").number("eps");
+    c.softcap = j.has("logit_softcap") ? (float)j.number("logit_softcap") : 0.0f;
+    if (c.vocab == 0 || c.width == 0) bad("vocab and width must be positive");
+    const Json& layers = j.at("layers");
+    if (layers.kind != Json::Array || layers.items.empty()) bad("'layers' is not a list of layers");
+    for (size_t i = 0; i < layers.items.size(); i++) {
+        const Json& e = layers.items[i];
+        LayerSpec l;
+        l.weights = i;
+        MixerSpec& m = l.mixer;
+        try {
+            const std::string& type = e.string("type");
+            const Json& x = e.at("mixer");
+            m.heads = x.size("heads");
+            m.dim = x.size("dim");
+            if (type == "gla") {
+                m.kind = MixerKind::Gla;
+                m.vdim = x.size("vdim");
+                m.tau = (float)x.number("tau");
+                if (!(m.tau > 0.0f)) bad("'tau' must be positive");
+            } else if (type == "wkv") {
+                m.kind = MixerKind::Wkv;
+                m.vdim = m.dim;
+            } else if (type == "latent_attention") {
+                m.kind = MixerKind::Latent;
+                m.vdim = x.size("vdim");
+                m.q_rank = x.size("q_rank");
+                m.kv_rank = x.size("kv_rank");
+                m.rot_dim = x.size("rot_dim");
+                m.scale = (float)x.number("scale");
+                const Json& rot = x.at("rot");
+                m.rot_base = rot.number("base");
+                m.rot_dims = rot.size("dims");
+                if (m.rot_dims % 2 || m.rot_dims > m.rot_dim) bad("'rot.dims' must be even and at most rot_dim");
+                if (x.has("mask")) {
+                    m.window = x.at("mask").size("size");
+                    if (m.window == 0) bad("'mask.size' must be positive");
+                }
+            } else {
+                bad("unknown mixer '" + type + "'");
+            }
+            if (m.heads == 0 || m.dim == 0 || m.vdim == 0) bad("head counts and sizes must be positive");
+            if (e.has("mlp")) {
+                const std::string& kind = e.at("mlp").string("kind");
+                if (kind != "dense") bad("unknown feed-forward '" + kind + "'");
+                l.ff = e.at("mlp").size("ff");
+                if (l.ff == 0) bad("'ff' must be positive");
+            }
+            if (e.has("weights_of")) {
+                l.weights = e.size("weights_of");
+                if (l.weights >= layers.items.size()) bad("'weights_of' names no layer");
+            }
+        } catch (const std::exception& ex) {
+            bad("layer " + std::to_string(i) + ": " + ex.what());
+        }
+        c.layers.push_back(l);
+    }
+    for (size_t i = 0; i < c.layers.size(); i++) {
+        size_t o = c.layers[i].weights;
+        for (size_t hops = 0; c.layers[o].weights != o; o = c.layers[o].weights)
+            if (++hops > c.layers.size()) bad("layer " + std::to_string(i) + ": 'weights_of' goes in a circle");
+        const LayerSpec& own = c.layers[o];
+        const MixerSpec &n = own.mixer, &m = c.layers[i].mixer;
+        if (n.kind != m.kind || n.heads != m.heads || n.dim != m.dim || n.vdim != m.vdim || n.q_rank != m.q_rank ||
+            n.kv_rank != m.kv_rank || n.rot_dim != m.rot_dim || own.ff != c.layers[i].ff)
+            bad("layer " + std::to_string(i) + ": 'weights_of' names a layer of other sizes");
+        c.layers[i].weights = o;
+    }
+    return c;
+}
+
+// ---------------------------------------------------------------------------------------------------- tensor sources
+namespace {
+struct FileSource : TensorSource {
+    std::shared_ptr<SafeTensors> f;
+    const SafeTensor& get(const std::string& name) {
+        const SafeTensor* t = f->find(name);
+        if (!t) bad("missing tensor " + name);
+        return *t;
+    }
+    void matrix(const std::string& name, size_t rows, size_t cols, uint16_t* out) override {
+        const SafeTensor& t = get(name);
+        if (t.shape != std::vector<size_t>{rows, cols})
+            bad(name + ": expected a " + std::to_string(rows) + " x " + std::to_string(cols) + " matrix");
+        if (t.dtype != "BF16") bad(name + ": expected bfloat16, found " + t.dtype);
+        std::memcpy(out, t.data, t.bytes);
+        for (size_t i = 0; i < rows * cols; i++)
+            if ((out[i] & 0x7F80) == 0x7F80) bad(name + ": not finite");
+    }
+    std::vector<float> vector(const std::string& name, size_t n) override {
+        const SafeTensor& t = get(name);
+        if (t.n_elems() != n) bad(name + ": expected " + std::to_string(n) + " values");
+        std::vector<float> v(n);
+        if (t.dtype == "F32") std::memcpy(v.data(), t.data, t.bytes);
+        else if (t.dtype == "BF16")
+            for (size_t i = 0; i < n; i++) {
+                uint16_t b;
+                std::memcpy(&b, t.data + 2 * i, 2);
+                v[i] = bf16_to_f32(b);
+            }
+        else bad(name + ": expected bfloat16 or float32, found " + t.dtype);
+        for (float x : v)
+            if (!std::isfinite(x)) bad(name + ": not finite");
+        return v;
+    }
+    size_t rows_of(const std::string& name, size_t cols) override {
+        const SafeTensor& t = get(name);
+        if (t.shape.size() != 2 || t.shape[1] != cols) bad(name + ": expected a matrix of width " + std::to_string(cols));
+        return t.shape[0];
+    }
+};
+struct SynthSource : TensorSource {
+    Backend* bk;
+    uint64_t seed, next = 1;
+    size_t rank = 64;      // of the low-rank decay projections
+    void matrix(const std::string&, size_t rows, size_t cols, uint16_t* out) override {
+        const uint64_t tid = next++;
+        for (size_t i = 0; i < rows * cols; i++) out[i] = f32_to_bf16(draw_normal(seed, tid, i, WEIGHT_STD));
+    }
+    std::vector<float> vector(const std::string& name, size_t n) override {
+        // unit norms; the small vectors of the mixers (mixes, biases, bonuses, sinks) are drawn
+        const bool norm = name.find("norm") != std::string::npos;
+        const uint64_t tid = next++;
+        std::vector<float> v(n, 1.0f);
+        if (!norm)
+            for (size_t i = 0; i < n; i++) v[i] = draw_unit(seed, tid, i);
+        return v;
+    }
+    size_t rows_of(const std::string&, size_t) override { return rank; }
+    bool on_device(const std::string&, size_t rows, size_t cols, uint16_t* out) override {
+        bk->synth_bf16(seed, next++, rows * cols, out);
+        return true;
+    }
+};
+
+// Rows of a packed linear: tensor rows go to given physical rows (stride `step`) at a column offset.
+class Packer {
+  public:
+    Packer(Backend* bk, TensorSource& src, size_t n, size_t k) : bk_(bk), src_(src) {
+        lin_.n = n;
+        lin_.k = k;
+        lin_.ld = round8(k);
+        lin_.w = bk->alloc<uint16_t>(n * lin_.ld);   // zero-filled
+    }
+    void part(const std::string& name, size_t rows, size_t cols, size_t row0, size_t step = 1, size_t col0 = 0) {
+        if (step == 1 && cols == lin_.ld && src_.on_device(name, rows, cols, lin_.w.ptr_at(row0 * lin_.ld))) return;
+        tmp_.resize(rows * cols);
+        src_.matrix(name, rows, cols, tmp_.data());
+        if (host_.empty()) host_.assign(lin_.n * lin_.ld, 0);
+        for (size_t r = 0; r < rows; r++)
+            std::memcpy(&host_[(row0 + r * step) * lin_.ld + col0], &tmp_[r * cols], cols * 2);
+        filled_.push_back({row0, step, rows});
+    }
+    FLinear finish() {
+        if (!host_.empty()) {
+            size_t lo = lin_.n, hi = 0;   // rows written on the host form one span (device-filled parts lie outside it)
+            for (const auto& f : filled_) {
+                lo = std::min(lo, f[0]);
+                hi = std::max(hi, f[0] + (f[2] - 1) * f[1] + 1);
+            }
+            bk_->write(lin_.w, lo * lin_.ld, host_.data() + lo * lin_.ld, (hi - lo) * lin_.ld);
+            bk_->sync();   // the staging buffer dies here
+        }
+        return std::move(lin_);
+    }
+
+  private:
+    Backend* bk_;
+    TensorSource& src_;
+    FLinear lin_;
+    std::vector<uint16_t> host_, tmp_;
+    std::vector<std::array<size_t, 3>> filled_;
+};
+}  // namespace
+
+// ---------------------------------------------------------------------------------------------------- loading
+static std::shared_ptr<HybridWeights> load_layer(const HybridConfig& c, size_t i, TensorSource& src, Backend* bk, bool synthetic) {
+    auto wp = std::make_shared<HybridWeights>();
+    HybridWeights& w = *wp;
+    const LayerSpec& l = c.layers[i];
+    const MixerSpec& m = l.mixer;
+    const std::string p = "l" + std::to_string(i) + ".", mix = p + "mix.", mlp = p + "mlp.";
+    const size_t W = c.width, qk = m.heads * m.dim, vo = m.width_out();
+    auto vec = [&](const std::string& name, size_t n) { return bk->upload(src.vector(name, n)); };
+    w.norm1 = vec(p + "norm1", W);
+
+    struct Part {
+        std::string name;
+        size_t rows;
+    };
+    std::vector<Part> parts;
+    switch (m.kind) {
+        case MixerKind::Gla:
+            w.rank = src.rows_of(mix + "a1", W);
+            parts = {{"q", qk}, {"k", qk}, {"v", vo}, {"g", vo}, {"a1", w.rank}};
+            break;
+        case MixerKind::Wkv:
+            w.rank = src.rows_of(mix + "w1", W);
+            parts = {{"r", qk}, {"k", qk}, {"v", vo}, {"g", vo}, {"w1", w.rank}};
+            break;
+        case MixerKind::Latent:
+            parts = {{"dq", m.q_rank}, {"dkv", m.kv_rank + m.rot_dim}, {"g", vo}};
+            break;
+    }
+    for (size_t q = 0; q < parts.size(); q++) {
+        w.off[q] = w.plain;
+        w.plain += parts[q].rows;
+    }
+    Packer in(bk, src, w.plain + 2 * l.ff, W);
+    for (size_t q = 0; q < parts.size(); q++) in.part(mix + parts[q].name, parts[q].rows, W, w.off[q]);
+    if (l.ff) {
+        if (synthetic && W % 8 == 0) {
+            in.part(mlp + "gate", 2 * l.ff, W, w.plain);   // a random matrix needs no interleaving
+        } else {
+            in.part(mlp + "gate", l.ff, W, w.plain, 2);
+            in.part(mlp + "up", l.ff, W, w.plain + 1, 2);
+        }
+    }
+    w.in = in.finish();
+
+    w.out_ff = round8(vo);
+    Packer out(bk, src, W, l.ff ? w.out_ff + l.ff : vo);
+    if (synthetic && vo % 8 == 0 && l.ff % 8 == 0) {
+        out.part(mix + "o", W, vo + l.ff, 0);
+    } else {
+        out.part(mix + "o", W, vo, 0);
+        if (l.ff) out.part(mlp + "down", W, l.ff, 0, 1, w.out_ff);
+    }
+    w.out = out.finish();
+
+    if (m.kind == MixerKind::Latent) {
+        w.dq_norm = vec(mix + "dq.norm", m.q_rank);
+        w.dkv_norm = vec(mix + "dkv.norm", m.kv_rank);
+        w.sink = vec(mix + "sink", m.heads);
+        Packer uq(bk, src, m.heads * (m.dim + m.rot_dim), m.q_rank);
+        uq.part(mix + "uq", m.heads * (m.dim + m.rot_dim), m.q_rank, 0);
+        w.uq = uq.finish();
+        Packer ukv(bk, src, qk + vo, m.kv_rank);
+        ukv.part(mix + "uk", qk, m.kv_rank, 0);
+        ukv.part(mix + "uv", vo, m.kv_rank, qk);
+        w.ukv = ukv.finish();
+        return wp;
+    }
+    const bool gla = m.kind == MixerKind::Gla;
+    Packer decay(bk, src, qk, w.rank);
+    decay.part(mix + (gla ? "a2" : "w2"), qk, w.rank, 0);
+    w.decay = decay.finish();
+    w.decay_bias = vec(mix + (gla ? "a2.b" : "w0"), qk);
+    if (gla) {
+        // one norm weight for all heads: repeated, so that the kernels index by channel in either mixer
+        const std::vector<float> n = src.vector(mix + "norm", m.vdim);
+        std::vector<float> all;
+        for (size_t h = 0; h < m.heads; h++) all.insert(all.end(), n.begin(), n.end());
+        w.head_norm = bk->upload(all);
+        bk->sync();
+    } else {
+        w.head_norm = vec(mix + "norm", vo);
+        w.bonus = vec(mix + "u", qk);
+        std::vector<float> mu;
+        for (const char* n : {"r", "k", "v", "g", "w"}) {
+            const std::vector<float> v = src.vector(mix + "mu." + n, W);
+            mu.insert(mu.end(), v.begin(), v.end());
+        }
+        w.mu = bk->upload(mu);
+        bk->sync();
+    }
+    return wp;
+}
+
+static HybridCache make_cache(const HybridConfig& c, Backend* bk, Dtype dtype, size_t ctx, size_t max_batch) {
+    HybridCache s;
+    for (const LayerSpec& l : c.layers) {
+        const MixerSpec& m = l.mixer;
+        FloatState f;
+        if (m.kind == MixerKind::Latent) {
+            // a step of max_batch tokens still needs the window before its first one
+            f.cap = m.window ? std::min(ctx, m.window - 1 + max_batch) : ctx;
+            f.cache = bk->alloc<uint8_t>(f.cap * (size_t)det_f_latent_ld((int)m.kv_rank, (int)m.rot_dim) * dtype_bytes(dtype));
+        } else {
+            f.s = bk->alloc<float>(m.heads * m.dim * m.vdim);
+            if (m.kind == MixerKind::Wkv) f.prev = bk->alloc<float>(c.width);
+        }
+        s.layers.push_back(std::move(f));
+    }
+    return s;
+}
+
+std::unique_ptr<HybridModel> HybridModel::load(const HybridConfig& cfg, TensorSource& src, Backend* bk, size_t max_ctx,
+                                               size_t max_batch, Dtype dtype) {
+    if (max_ctx == 0 || max_batch == 0) bad("the context and the batch must be positive");
+    auto mp = std::make_unique<HybridModel>();
+    HybridModel& m = *mp;
+    m.cfg = cfg;
+    m.backend = bk;
+    m.dtype = dtype;
+    m.max_ctx = max_ctx;
+    m.max_batch = max_batch;
+    const bool synthetic = dynamic_cast<SynthSource*>(&src) != nullptr;
+    const size_t W = cfg.width;
+    {
+        std::vector<uint16_t> e(cfg.vocab * W);
+        src.matrix("embed", cfg.vocab, W, e.data());
+        m.embed_ = bk->upload(e);
+        bk->sync();
+    }
+    m.weights_.resize(cfg.layers.size());
+    for (size_t i = 0; i < cfg.layers.size(); i++)
+        if (cfg.layers[i].weights == i) m.weights_[i] = load_layer(cfg, i, src, bk, synthetic);
+    for (size_t i = 0; i < cfg.layers.size(); i++) m.weights_[i] = m.weights_[cfg.layers[i].weights];
+    m.final_norm_ = bk->upload(src.vector("final.norm", W));
+    bk->sync();
+    Packer head(bk, src, cfg.vocab, W);
+    head.part("head", cfg.vocab, W, 0);
+    m.head_lin_ = head.finish();
+
+    for (const LayerSpec& l : cfg.layers) {
+        const MixerSpec& x = l.mixer;
+        if (x.kind != MixerKind::Latent || std::any_of(m.ropes_.begin(), m.ropes_.end(), [&](const Rope& r) {
+                return r.base == x.rot_base && r.dims == x.rot_dims;
+            }))
+            continue;
+        const size_t half = x.rot_dims / 2;
+        std::vector<float> rc(max_ctx * half + 1), rs(max_ctx * half + 1);
+        for (size_t p = 0; p < max_ctx; p++)
+            for (size_t i = 0; i < half; i++) {
+                const double a = (double)p * std::pow(x.rot_base, -2.0 * (double)i / (double)x.rot_dims);
+                rc[p * half + i] = (float)std::cos(a);
+                rs[p * half + i] = (float)std::sin(a);
+            }
+        m.ropes_.push_back(Rope{x.rot_base, x.rot_dims, bk->upload(rc), bk->upload(rs)});
+        bk->sync();
+    }
+    m.bound_ = make_cache(cfg, bk, dtype, max_ctx, max_batch);
+
+    size_t groups = 1, ldy = 1, cat = 8, q = 1;
+    m.ld_cq_ = 8;
+    for (size_t i = 0; i < cfg.layers.size(); i++) {
+        const HybridWeights& w = *m.weights_[i];
+        const MixerSpec& x = cfg.layers[i].mixer;
+        ldy = std::max(ldy, w.plain);
+        cat = std::max(cat, w.out.ld);
+        if (x.kind == MixerKind::Wkv) groups = 6;
+        if (x.kind == MixerKind::Latent) {
+            m.ld_cq_ = std::max(m.ld_cq_, round8(x.q_rank));
+            q = std::max(q, x.heads * (x.dim + x.rot_dim));
+        }
+    }
+    m.ld_in_ = round8(W);
+    const size_t e = dtype_bytes(dtype);
+    m.in_ = bk->alloc<uint8_t>(groups * max_batch * m.ld_in_ * e);
+    m.cat_ = bk->alloc<uint8_t>(max_batch * cat * e);
+    m.cq_ = bk->alloc<uint8_t>(max_batch * m.ld_cq_ * e);
+    m.y_ = bk->alloc<float>(max_batch * ldy);
+    m.q_ = bk->alloc<float>(max_batch * q);
+    m.ids_ = bk->alloc<int32_t>(max_batch);
+    m.rows_ = bk->alloc<int32_t>(max_batch);
+    m.x = bk->alloc<float>(max_batch * W);
+    m.logits_buf = bk->alloc<float>(cfg.vocab);
+    return mp;
+}
+
+std::unique_ptr<HybridModel> HybridModel::load_dir(const std::string& dir, const Json& config, Backend* bk, size_t max_ctx,
+                                                   size_t max_batch, Dtype dtype) {
+    FileSource src;
+    src.f = SafeTensors::open(dir + "/model.safetensors");
+    return load(HybridConfig::from_json(config), src, bk, max_ctx, max_batch, dtype);
+}
+std::unique_ptr<HybridModel> HybridModel::load_synthetic(const Json& config, uint64_t seed, Backend* bk, size_t max_ctx,
+                                                         size_t max_batch, Dtype dtype) {
+    SynthSource src;
+    src.bk = bk;
+    src.seed = seed;
+    return load(HybridConfig::from_json(config), src, bk, max_ctx, max_batch, dtype);
+}
+
+size_t HybridModel::weight_bytes() const {
+    auto bytes = [](const FLinear& l) { return l.n * l.ld * 2; };
+    size_t s = bytes(head_lin_);
+    for (const auto& w : weights_) s += bytes(w->in) + bytes(w->out) + bytes(w->decay) + bytes(w->uq) + bytes(w->ukv);
+    return s;
+}
+
+// ---------------------------------------------------------------------------------------------------- sequences
+std::unique_ptr<SeqCache> HybridModel::new_sequence(size_t ctx) {
+    if (ctx > max_ctx) bad("a sequence's context exceeds the model's");   // the rotation tables end there
+    return std::make_unique<HybridCache>(make_cache(cfg, backend, dtype, ctx, max_batch));
+}
+void HybridModel::swap_sequence(SeqCache& s) { std::swap(bound_.layers, dynamic_cast<HybridCache&>(s).layers); }
+// Cache rows need no clearing: a position only reads rows its own sequence wrote.
+void HybridModel::clear_sequence(SeqCache& s) {
+    for (FloatState& f : dynamic_cast<HybridCache&>(s).layers) {
+        if (f.s.ptr()) backend->zero(f.s);
+        if (f.prev.ptr()) backend->zero(f.prev);
+    }
+}
+std::vector<std::unique_ptr<RowSet>> HybridModel::make_rowsets(const std::vector<SeqCache*>& seqs) {
+    std::vector<std::unique_ptr<RowSet>> sets;
+    for (size_t i = 0; i < cfg.layers.size(); i++) {
+        std::vector<const FloatState*> fs;
+        for (SeqCache* s : seqs) {
+            fs.push_back(&dynamic_cast<HybridCache&>(*s).layers[i]);
+            if (fs.back()->cap != fs[0]->cap) bad("the sequences of a batch must have caches of one size");
+        }
+        sets.push_back(backend->make_slots(std::move(fs)));
+    }
+    return sets;
+}
+
+// ---------------------------------------------------------------------------------------------------- network
+std::string HybridModel::embed_rows(const int32_t* ids, size_t t) {
+    for (size_t i = 0; i < t; i++)
+        if (ids[i] < 0 || (size_t)ids[i] >= cfg.vocab)
+            return "token id " + std::to_string(ids[i]) + " is outside the embedding table (" + std::to_string(cfg.vocab) + " rows)";
+    backend->write(ids_, 0, ids, t);
+    backend->embed(embed_.ptr(), 30, ids_, t, cfg.width, x);
+    return "";
+}
+
+const HybridModel::Rope& HybridModel::rope(const MixerSpec& m) const {
+    for (const Rope& r : ropes_)
+        if (r.base == m.rot_base && r.dims == m.rot_dims) return r;
+    throw std::logic_error("no rotation table");
+}
+
+// norm1 and every projection of the normalised row: mixer parts into y_, SwiGLU product behind the mixer's columns of cat_
+void HybridModel::run_in(const LayerSpec& l, const HybridWeights& w, size_t t, const det_seq_ref& seq) {
+    const det_flinear lin = w.in.view();
+    det_fgemm_op g{};
+    g.lin = &lin;
+    g.dtype = (int)dtype;
+    g.x = in_.ptr();
+    g.ldx = (int)ld_in_;
+    g.group_stride = (long long)(max_batch * ld_in_);
+    g.M = (int)t;
+    g.glu_from = (int)w.plain;
+    auto segment = [&](size_t end, int in) {
+        g.seg_end[g.nseg] = (int)end;
+        g.seg_in[g.nseg++] = in;
+    };
+    if (l.mixer.kind == MixerKind::Wkv) {
+        det_fnorm_op n{};
+        n.x = x.ptr();
+        n.w = w.norm1.ptr();
+        n.eps = cfg.eps;
+        n.M = (int)t;
+        n.n = (int)cfg.width;
+        n.dtype = (int)dtype;
+        n.out = in_.ptr();
+        n.ld = (int)ld_in_;
+        n.group_stride = g.group_stride;
+        n.nmix = 5;
+        n.mu = w.mu.ptr();
+        n.seq = seq;
+        backend->f_norm(n);
+        for (int p = 0; p < 5; p++) segment(p < 4 ? w.off[p + 1] : w.plain, p);
+        if (l.ff) segment(w.in.n, 5);
+    } else {
+        g.norm_x = x.ptr();
+        g.norm_w = w.norm1.ptr();
+        g.eps = cfg.eps;
+        segment(w.plain, 0);
+        if (l.ff) segment(w.in.n, 0);
+    }
+    g.y = y_.ptr();
+    g.ldy = (int)w.plain;
+    g.h = cat_.ptr() + w.out_ff * dtype_bytes(dtype);
+    g.ldh = (int)w.out.ld;
+    backend->f_gemm(g);
+}
+
+void HybridModel::mixer_recurrent(const LayerSpec& l, const HybridWeights& w, size_t t, const det_seq_ref& seq) {
+    const MixerSpec& m = l.mixer;
+    const det_flinear w2 = w.decay.view();
+    const bool gla = m.kind == MixerKind::Gla;
+    det_frecur_op r{};
+    r.heads = (int)m.heads;
+    r.dk = (int)m.dim;
+    r.dv = (int)m.vdim;
+    r.rank = (int)w.rank;
+    r.M = (int)t;
+    r.dtype = (int)dtype;
+    r.y = y_.ptr();
+    r.ldy = (int)w.plain;
+    r.q_off = (int)w.off[0];
+    r.k_off = (int)w.off[1];
+    r.v_off = (int)w.off[2];
+    r.gate_off = (int)w.off[3];
+    r.low_off = (int)w.off[4];
+    r.q_scale = gla ? (float)(1.0 / std::sqrt((double)m.dim)) : 1.0f;
+    r.decay = gla ? DET_DECAY_SIGMOID : DET_DECAY_EXP;
+    r.tau = m.tau;
+    r.w2 = &w2;
+    r.bias = w.decay_bias.ptr();
+    r.u = gla ? nullptr : w.bonus.ptr();
+    r.norm = w.head_norm.ptr();
+    r.eps = cfg.eps;
+    r.out = cat_.ptr();
+    r.ldo = (int)w.out.ld;
+    r.seq = seq;
+    backend->f_recur(r);
+}
+
+void HybridModel::mixer_latent(const LayerSpec& l, const HybridWeights& w, size_t t, const det_seq_ref& seq, size_t cap, size_t max_pos) {
+    const MixerSpec& m = l.mixer;
+    const det_flinear uq = w.uq.view(), ukv = w.ukv.view();
+    const Rope& rp = rope(m);
+    det_flatent_op a{};
+    a.heads = (int)m.heads;
+    a.dim = (int)m.dim;
+    a.rot_dim = (int)m.rot_dim;
+    a.rot_dims = (int)m.rot_dims;
+    a.vdim = (int)m.vdim;
+    a.q_rank = (int)m.q_rank;
+    a.kv_rank = (int)m.kv_rank;
+    a.window = (int)m.window;
+    a.scale = m.scale;
+    a.cap = (int)cap;
+    a.M = (int)t;
+    a.dtype = (int)dtype;
+    a.y = y_.ptr();
+    a.ldy = (int)w.plain;
+    a.dq_off = (int)w.off[0];
+    a.dkv_off = (int)w.off[1];
+    a.gate_off = (int)w.off[2];
+    a.dq_norm = w.dq_norm.ptr();
+    a.dkv_norm = w.dkv_norm.ptr();
+    a.eps = cfg.eps;
+    a.rope_cos = rp.cos.ptr();
+    a.rope_sin = rp.sin.ptr();
+    a.cq = cq_.ptr();
+    a.ldcq = (int)ld_cq_;
+    a.q = q_.ptr();
+    a.ldq = (int)w.uq.n;
+    a.wkv = &ukv;
+    a.sink = w.sink.ptr();
+    a.out = cat_.ptr();
+    a.ldo = (int)w.out.ld;
+    a.max_pos = (int)max_pos;
+    a.seq = seq;
+    backend->f_latent_prep(a);
+    det_fgemm_op g{};
+    g.lin = &uq;
+    g.dtype = (int)dtype;
+    g.x = cq_.ptr();
+    g.ldx = (int)ld_cq_;
+    g.nseg = 1;
+    g.seg_end[0] = (int)w.uq.n;
+    g.glu_from = (int)w.uq.n;
+    g.M = (int)t;
+    g.y = q_.ptr();
+    g.ldy = (int)w.uq.n;
+    backend->f_gemm(g);
+    backend->f_latent_attn(a, max_ctx);
+}
+
+// final norm, output rows, soft cap
+void HybridModel::head(size_t t) {
+    const det_flinear lin = head_lin_.view();
+    det_fgemm_op g{};
+    g.lin = &lin;
+    g.dtype = (int)dtype;
+    g.x = in_.ptr();
+    g.ldx = (int)ld_in_;
+    g.nseg = 1;
+    g.seg_end[0] = (int)cfg.vocab;
+    g.glu_from = (int)cfg.vocab;
+    g.y = logits_buf.ptr();
+    g.ldy = (int)cfg.vocab;
+    g.softcap = cfg.softcap;
+    g.norm_x = all_logits ? x.ptr() : x.ptr_at((t - 1) * cfg.width);
+    g.norm_w = final_norm_.ptr();
+    g.eps = cfg.eps;
+    g.M = all_logits ? (int)t : 1;
+    if (head_rows_) {
+        if (head_rows_->empty()) return;
+        backend->write(rows_, 0, head_rows_->data(), head_rows_->size());
+        det_fnorm_op n{};
+        n.x = x.ptr();
+        n.rows = rows_.ptr();
+        n.w = final_norm_.ptr();
+        n.eps = cfg.eps;
+        n.M = g.M = (int)head_rows_->size();
+        n.n = (int)cfg.width;
+        n.dtype = (int)dtype;
+        n.out = in_.ptr();
+        n.ld = (int)ld_in_;
+        backend->f_norm(n);
+        g.norm_x = nullptr;
+    }
+    backend->f_gemm(g);
+}
+
+void HybridModel::network(size_t pos0, size_t t, Observer* obs, const RowsCtx* rows) {
+    if (obs && rows) throw std::logic_error("observers are not supported on a batched decode step");
+    if (head_rows_ && head_rows_->size() > max_batch) throw std::logic_error("more logits rows than the batch holds");
+    const Ctx ctx{pos0, t, backend};
+    auto observe = [&](Tap::Kind kind, size_t layer, const Buf<float>& b) {
+        if (!obs) return;
+        Tap tap;
+        tap.kind = kind;
+        tap.layer = layer;
+        tap.x = &b;
+        obs->observe(ctx, tap);
+    };
+    const size_t max_pos = rows ? rows->max_pos : pos0 + t - 1;
+    for (size_t li = 0; li < cfg.layers.size(); li++) {
+        observe(Tap::Residual, li, x);
+        const LayerSpec& l = cfg.layers[li];
+        const HybridWeights& w = *weights_[li];
+        const RowSet* set = rows ? (*rows->sets)[li].get() : nullptr;
+        const FloatState& state = set ? *set->fs[0] : bound_.layers[li];
+        const det_seq_ref seq = backend->seq_ref(state, pos0, set, rows ? rows->pos : nullptr);
+        run_in(l, w, t, seq);
+        if (l.mixer.kind == MixerKind::Latent) mixer_latent(l, w, t, seq, state.cap, max_pos);
+        else mixer_recurrent(l, w, t, seq);
+        const det_flinear out = w.out.view();
+        det_fgemm_op g{};
+        g.lin = &out;
+        g.dtype = (int)dtype;
+        g.x = cat_.ptr();
+        g.ldx = (int)w.out.ld;
+        g.nseg = 1;
+        g.seg_end[0] = (int)cfg.width;
+        g.glu_from = (int)cfg.width;
+        g.M = (int)t;
+        g.y = x.ptr();
+        g.ldy = (int)cfg.width;
+        g.accumulate = 1;
+        backend->f_gemm(g);
+    }
+    observe(Tap::Residual, cfg.layers.size(), x);
+    head(t);
+    observe(Tap::Logits, 0, logits_buf);
+}
+
+}  // namespace det

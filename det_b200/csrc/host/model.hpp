@@ -1,13 +1,12 @@
-// The model, its activation buffers and the token loop — the C++ mirror of crates/det/src/model.rs (Proj, Attn, Gdn,
-// Layer, Work, Sampling, Model::{load, set_all_logits, reset, embed_rows, project, forward, logits, pick, prefill,
-// generate}) and of the network's op sequence crates/det/src/qwen35.rs:8-172.  It talks to a backend only through
-// the op set of backend.hpp, so the same driver runs the CUDA backend and, in tests, the CPU reference backend.
+// What every model shares: the token loop (embed, forward, prefill, pick, generate) and the handling of per-sequence caches —
+// the C++ mirror of the model-independent part of crates/det/src/model.rs (Sampling, Model::{set_all_logits, reset, forward,
+// logits, pick, prefill, generate}).  A concrete model (qwen35.hpp, hybrid.hpp) supplies its network and its caches; the
+// batched decoder (serve.hpp), the graph decoder (graph_decode.hpp) and the C entry points work on this interface.  A model
+// talks to a backend only through the op set of backend.hpp.
 #pragma once
 #include "backend.hpp"
 #include "comm.hpp"
-#include "gguf.hpp"
 #include "hooks.hpp"
-#include "synth.hpp"
 #include <functional>
 #include <memory>
 #include <string>
@@ -15,54 +14,18 @@
 
 namespace det {
 
-constexpr float DEFAULT_V_SCALE = 1.0f / 1024.0f;   // model.rs:47
-
-struct Proj {   // model.rs:51-53
-    std::vector<std::unique_ptr<Linear>> lins;
-};
-struct Attn {   // model.rs:55-63
-    Proj qkv, o;
-    Buf<float> q_norm, k_norm, v_scale, v_inv_scale;
-    KvCache kv;
-};
-struct Gdn {   // model.rs:65-74
-    Proj qkvz, ab, out;
-    Buf<float> conv, a, dt_bias, norm;
-    GdnState state;
-};
-struct Layer {   // model.rs:81-87
-    Buf<float> attn_norm, ffn_norm;
-    Proj gu, down;
-    bool is_attn = false;
-    Attn attn;
-    Gdn gdn;
-};
-struct Work {   // model.rs:89-118
-    Buf<float> x;
-    Buf<int8_t> xq;
-    Buf<float> sx;
-    Buf<uint16_t> mx;
-    Buf<float> qg, k, v, o;
-    Buf<int8_t> oq;
-    Buf<float> so;
-    Buf<uint16_t> mo;
-    Buf<float> qkv, z, a, b, on;
-    Buf<int8_t> onq;
-    Buf<float> son;
-    Buf<uint16_t> mon;
-    Buf<float> g, u;
-    Buf<int8_t> hq;
-    Buf<float> sh;
-    Buf<uint16_t> mh;
-    Buf<float> logits;
-    Buf<float> gin, gout;   // GDN mixer export (model.rs:343-344); sized on the first observed step that asks for them
-};
 struct Sampling {   // model.rs:120-141
     bool greedy = true;
     float inv_temp = 1.0f;
     size_t top_k = 0;
     float top_p = 1.0f;
     uint64_t rng = 0;
+};
+
+// Everything one sequence keeps between steps, in every layer (a key/value cache, a recurrent state, ...).  A model makes
+// them for as many sequences as a caller holds; exactly one is bound to the model at a time.
+struct SeqCache {
+    virtual ~SeqCache() = default;
 };
 
 // The per-sequence caches / states behind the rows of a batched decode step (serve.hpp): with it the network takes row b
@@ -73,26 +36,39 @@ struct RowsCtx {
     size_t max_pos;                                     // host bound on the positions
 };
 
+// The embedding table in backend memory, for steps whose token comes from the device.
+struct EmbedTable {
+    const void* table = nullptr;
+    int type = 30;   // ggml type: 0 F32, 1 F16, 30 BF16
+};
+
 class Model {
   public:
-    // A seeded random-init model of shape `cfg` (the stand-in for Model::load on a converted checkpoint).
-    // `comm` (optional) makes this the shard of rank comm->rank in a tensor-parallel group of comm->size: linears are
-    // cut by output rows, attention by q heads, Gated DeltaNet by k heads, the FFN by 128-column groups, the head by
-    // vocabulary rows; the residual stream and the norms stay replicated (see network_tp in model.cpp).
-    static std::unique_ptr<Model> load_synthetic(const Config& cfg, uint64_t seed, Backend* backend, size_t max_ctx,
-                                                 size_t max_batch, Comm* comm = nullptr);
+    virtual ~Model() = default;
+    Model() = default;
+    Model(const Model&) = delete;
+    Model& operator=(const Model&) = delete;
 
-    // Model::load (model.rs:164-365): a det GGUF written by `det convert` (or write_synthetic_gguf).  Null and a message in
-    // `err` when the file is unreadable, not a qwen35 det file, holds a non-finite value, or lacks a tensor.
-    static std::unique_ptr<Model> load(const std::string& path, Backend* backend, size_t max_ctx, size_t max_batch,
-                                       std::string& err);
+    virtual size_t vocab() const = 0;
+    virtual size_t hidden() const = 0;
+    // Residual rows of `t` tokens into x; "" on success (model.rs:389-413).
+    virtual std::string embed_rows(const int32_t* ids, size_t t) = 0;
+    // The network over the `t` rows of x: positions pos0 .. pos0 + t of the bound sequence, or one row per sequence with
+    // `rows`.  Leaves logits in logits_buf: of the rows named by forward_rows(), of every row when all_logits, else of the last.
+    virtual void network(size_t pos0, size_t t, Observer* obs = nullptr, const RowsCtx* rows = nullptr) = 0;
+
+    // ---- caches of further sequences
+    virtual std::unique_ptr<SeqCache> new_sequence(size_t ctx) = 0;      // room for ctx positions, cleared
+    virtual void swap_sequence(SeqCache& s) = 0;                          // exchanges the bound caches with these
+    virtual void clear_sequence(SeqCache& s) = 0;                         // back to position 0
+    virtual std::vector<std::unique_ptr<RowSet>> make_rowsets(const std::vector<SeqCache*>& seqs) = 0;   // one per layer
+    virtual EmbedTable embed_table() = 0;
 
     void set_all_logits(bool all);                                   // model.rs:367-375
     void reset();                                                    // model.rs:377-387
-    std::string embed_rows(const int32_t* ids, size_t t);            // model.rs:389-413; "" on success
-    void project(const Proj& p, const Buf<int8_t>& xq, const Buf<float>& sx, const Buf<uint16_t>& mx, size_t t,
-                 const std::vector<const Buf<float>*>& dsts);        // model.rs:415-437
     std::string forward(const int32_t* ids, size_t t, Observer* obs = nullptr);            // model.rs:439-465
+    // One step whose logits are wanted for the given rows (ascending or not, possibly none), in that order in logits_buf.
+    std::string forward_rows(const int32_t* ids, size_t t, const std::vector<int32_t>& want);
     std::vector<float> logits();                                     // model.rs:467-470
     std::string pick(Sampling& s, int32_t& id);                      // model.rs:472-496
     std::string pick_row(const Buf<float>& logits_row, Sampling& s, int32_t& id);   // the same draw on a given logits row
@@ -102,37 +78,16 @@ class Model {
                          const std::vector<int32_t>& stop, std::vector<int32_t>& out,
                          const std::function<void(int32_t)>& on_token = nullptr, Observer* obs = nullptr);   // model.rs:510-547
 
-    Config cfg;
     Backend* backend = nullptr;
-    uint64_t seed = 0;
-    std::shared_ptr<Gguf> gguf;   // the mapped file of a loaded model (null for a synthetic one); owns the embedding rows
-    GgufTensor embed;             // token_embd.weight of `gguf`
-    bool calibrated = false;      // the file carries value scales other than the default (model.rs:236-244)
-    Buf<float> final_norm, rope_cos, rope_sin;
-    Proj lm_head;
-    std::vector<Layer> layers;
-    Work w;
     size_t max_ctx = 0, max_batch = 0, pos = 0;
     bool all_logits = false;
+    Buf<float> x;            // residual rows [max_batch][hidden]
+    Buf<float> logits_buf;   // [vocab], or one row per requested position
 
-    void network(size_t pos0, size_t t, Observer* obs = nullptr, const RowsCtx* rows = nullptr);   // qwen35.rs:8-172
-
-    // ---- tensor parallel state (comm == nullptr: none of it is used)
-    Comm* comm = nullptr;
-    struct Tp {
-        size_t heads = 0, kv = 0;        // local q heads / kv heads of an attention layer
-        size_t k_heads = 0, v_heads = 0; // local GDN heads
-        size_t ffn = 0, hid = 0, voc = 0;   // local FFN columns, hidden rows, vocabulary rows
-        Buf<float> mix_full;   // [mb][n_h*hd] gathered mixer output
-        Buf<float> h_l, h_full;      // SwiGLU product, local and gathered
-        Buf<float> y_l, y_full;      // projection back to hidden, local rows and gathered
-        Buf<float> logits_l;
-        Buf<float> tmp;              // all-gather scratch
-        Buf<float> x_alt;            // second copy of the residual stream (an exchange fused into a GEMV stores the sums here)
-    } tp;
-
-  private:
-    void network_tp(size_t pos0, size_t t, const RowsCtx* rows);
+  protected:
+    virtual void clear_bound() = 0;                 // the bound sequence back to its start
+    virtual void logits_resized(size_t) {}
+    const std::vector<int32_t>* head_rows_ = nullptr;   // set while forward_rows() runs
 };
 
 }  // namespace det

@@ -7,51 +7,19 @@ namespace det {
 
 BatchDecoder::BatchDecoder(Model& model, size_t n_seq, size_t ctx) : seqs(n_seq), m_(model), ctx_(ctx) {
     if (n_seq == 0 || n_seq > model.max_batch) throw std::runtime_error("the model's max_batch is smaller than the number of sequences");
-    Backend* bk = model.backend;
-    const Config& c = model.cfg;
-    // a tensor-parallel shard keeps this rank's kv heads and GDN heads of every sequence (model.hpp, Model::Tp)
-    const size_t n_kv = model.comm ? model.tp.kv : c.n_kv;
-    const size_t k_heads = model.comm ? model.tp.k_heads : c.gdn_k_heads, v_heads = model.comm ? model.tp.v_heads : c.gdn_v_heads;
-    const size_t conv_dim = 2 * k_heads * c.gdn_dk + v_heads * c.gdn_dv;
+    std::vector<SeqCache*> caches;
     for (Sequence& s : seqs) {
-        for (const Layer& l : model.layers) {
-            if (l.is_attn) {
-                KvCache kv;   // model.rs:278-283
-                kv.kq = bk->alloc<int8_t>(ctx * n_kv * c.head_dim);
-                kv.sk = bk->alloc<float>(ctx * n_kv);
-                kv.vq = bk->alloc<int16_t>(ctx * n_kv * c.head_dim);
-                kv.capacity = ctx;
-                s.kv.push_back(std::move(kv));
-            } else {
-                GdnState st;   // model.rs:300-303
-                st.conv_state = bk->alloc<float>((c.conv_k - 1) * conv_dim);
-                st.s = bk->alloc<float>(v_heads * c.gdn_dk * c.gdn_dv);
-                s.st.push_back(std::move(st));
-            }
-        }
+        s.cache = model.new_sequence(ctx);
+        caches.push_back(s.cache.get());
     }
-    size_t ia = 0, ig = 0;
-    for (const Layer& l : model.layers) {
-        std::vector<const KvCache*> kv;
-        std::vector<const GdnState*> st;
-        for (Sequence& s : seqs) {
-            if (l.is_attn) kv.push_back(&s.kv[ia]);
-            else st.push_back(&s.st[ig]);
-        }
-        (l.is_attn ? ia : ig)++;
-        rowsets_.push_back(bk->make_rowset(std::move(kv), std::move(st)));
-    }
-    pos_ = bk->alloc<int32_t>(n_seq);
+    rowsets_ = model.make_rowsets(caches);
+    pos_ = model.backend->alloc<int32_t>(n_seq);
     model.set_all_logits(true);   // logits of every row of a step
 }
 
 void BatchDecoder::bind(size_t i) {
     Sequence& s = seqs[i];
-    size_t ia = 0, ig = 0;
-    for (Layer& l : m_.layers) {
-        if (l.is_attn) std::swap(l.attn.kv, s.kv[ia++]);
-        else std::swap(l.gdn.state, s.st[ig++]);
-    }
+    m_.swap_sequence(*s.cache);
     std::swap(m_.pos, s.pos);
 }
 
@@ -66,10 +34,7 @@ std::string BatchDecoder::prefill(size_t i, const int32_t* ids, size_t n, const 
     if (s.pos != 0) {
         m_.backend->sync();
         s.pos = 0;
-        for (GdnState& st : s.st) {
-            m_.backend->zero(st.conv_state);
-            m_.backend->zero(st.s);
-        }
+        m_.clear_sequence(*s.cache);
     }
     const size_t max_ctx = m_.max_ctx;
     m_.max_ctx = ctx_;
@@ -109,7 +74,7 @@ std::string BatchDecoder::step() {
     if (!e.empty()) return e;
     m_.backend->write(pos_, 0, pos.data(), t);
     network_rows(t);
-    const size_t v = m_.cfg.vocab;
+    const size_t v = m_.vocab();
     // all rows in one call when the sequences share their sampling parameters (each keeps its own generator)
     const Sampling& s0 = seqs[0].sampling;
     bool same = std::isfinite(s0.inv_temp) && !std::isnan(s0.top_p);
@@ -118,15 +83,15 @@ std::string BatchDecoder::step() {
                s.sampling.top_k == s0.top_k && s.sampling.top_p == s0.top_p;
     std::vector<int32_t> picked;
     if (same && s0.greedy) {
-        picked = m_.backend->argmax_rows(m_.w.logits, t, v);
+        picked = m_.backend->argmax_rows(m_.logits_buf, t, v);
     } else if (same) {
         std::vector<uint64_t> z(t);
         for (size_t b = 0; b < t; b++) z[b] = Model::next_draw(seqs[b].sampling);
-        picked = m_.backend->sample_rows(m_.w.logits, t, v, s0.inv_temp, s0.top_k, s0.top_p, z);
+        picked = m_.backend->sample_rows(m_.logits_buf, t, v, s0.inv_temp, s0.top_k, s0.top_p, z);
     } else {
         picked.resize(t);
         for (size_t b = 0; b < t; b++) {
-            e = m_.pick_row(Buf<float>::view(m_.w.logits.ptr_at(b * v), v), seqs[b].sampling, picked[b]);
+            e = m_.pick_row(Buf<float>::view(m_.logits_buf.ptr_at(b * v), v), seqs[b].sampling, picked[b]);
             if (!e.empty()) return e;
         }
     }

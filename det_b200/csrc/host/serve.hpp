@@ -11,8 +11,7 @@
 namespace det {
 
 struct Sequence {
-    std::vector<KvCache> kv;       // one per attention layer, in layer order
-    std::vector<GdnState> st;      // one per GDN layer, in layer order
+    std::unique_ptr<SeqCache> cache;   // made by the model: what its layers keep for one sequence
     size_t pos = 0;
     Sampling sampling;
     int32_t last = 0;              // the token that the next step feeds

@@ -375,6 +375,172 @@ void det_clear_error(void);
 void det_debug_set_wait_limit(long long cycles);
 void det_debug_xchg_drop(void* h, int rank);
 
+/* ================================================================================================================
+ * Part 3 — floating-point op set (no counterpart in the reference, whose models are integer-quantized)
+ *
+ * Ops of decoder models whose linears stay in bfloat16.  `dtype` names the type of the activations that enter a linear:
+ * DET_BF16 (tensor-core products, 32-bit accumulation) or DET_F32 (everything in 32-bit; a bfloat16 weight widens exactly).
+ * Residual rows, norms, scores, decays and recurrent state are fp32 either way.  Activation buffers of either type have a
+ * row stride that is a multiple of 8 elements, 16-byte aligned rows and zeros behind the last column.
+ * ============================================================================================================== */
+#define DET_F32 0
+#define DET_BF16 1
+
+/* W[N][ld] bfloat16, ld a multiple of 8, columns K..ld zero. */
+typedef struct {
+    const void* w;
+    int N, K, ld;
+} det_flinear;
+
+/* What one sequence keeps in one layer: recurrent state s[heads][dk][dv], the previous token's normalised row prev[n], and
+ * a cache of `cap` rows used as a ring (the row of position p is row p % cap).  A layer uses the members it needs.     */
+typedef struct {
+    float* s;
+    float* prev;
+    void* cache;
+} det_seq_slot;
+/* Which sequence and position the rows of a step belong to.  table == NULL: the rows are consecutive tokens of the sequence
+ * `one`, the first at position pos ? *pos : pos0 (pos: device word, so that a captured step can be replayed).
+ * table != NULL (device array): row r is the next token of the sequence table[r], at position pos[r] (device array).   */
+typedef struct {
+    const det_seq_slot* table;
+    det_seq_slot one;
+    const int* pos;
+    int pos0;
+} det_seq_ref;
+
+/* out[g][row][.] for g = nmix: h = x / sqrt(mean(x^2) + eps) * w; for g < nmix: h + (h' - h) * mu[g], h' being the
+ * normalised row of the token before (prev of the sequence for the first one), and prev receives the last h.
+ * rows != NULL (device): row r is taken from x row rows[r].  Group g starts at out + g * group_stride elements.         */
+typedef struct {
+    const float* x;
+    const int* rows;
+    const float* w;
+    float eps;
+    int M, n;
+    int dtype;
+    void* out;
+    int ld;
+    long long group_stride;
+    int nmix;
+    const float* mu;          /* [nmix][n] */
+    det_seq_ref seq;          /* only with nmix > 0 */
+} det_fnorm_op;
+void det_f_norm(const det_fnorm_op* op, cudaStream_t st);
+
+/* Y = X W^T over M rows, with its neighbours:
+ *   - the rows of W come in nseg segments, segment i ending before row seg_end[i]; its input is group seg_in[i] of x
+ *     (x + seg_in[i] * group_stride elements), so that linears over different inputs go out as one launch;
+ *   - norm_x != NULL (one group only): the input rows are the RMS norm of norm_x (norm_w, eps).  A decode-sized call
+ *     builds them in its prologue; a larger one runs det_f_norm into x first (x is then written);
+ *   - rows of W from glu_from on (a segment start, or N for none) are (gate, up) pairs: h[row][(n - glu_from) / 2] =
+ *     silu(gate) * up, in the activation type;
+ *   - rows before glu_from land in y[row][n] (fp32, or bfloat16 with y_bf16), added to it with `accumulate`;
+ *     softcap > 0: softcap * tanh(y / softcap).                                                                        */
+typedef struct {
+    const det_flinear* lin;
+    int dtype;
+    const void* x;
+    int ldx;
+    long long group_stride;
+    int nseg;
+    int seg_end[8];
+    int seg_in[8];
+    int glu_from;
+    int M;
+    const float* norm_x;
+    const float* norm_w;
+    float eps;
+    void* y;
+    int ldy;
+    int y_bf16;
+    int accumulate;
+    float softcap;
+    void* h;
+    int ldh;
+} det_fgemm_op;
+void det_f_gemm(const det_fgemm_op* op, cudaStream_t st);
+
+/* Linear recurrence with a decay per key channel, state S[dk][dv] per head:
+ *   S <- diag(decay) S + k v^T ; o = S^T q                       (u == NULL: the read follows the update)
+ *   o = (S + diag(u) k v^T)^T q ; S <- diag(decay) S + k v^T      (u != NULL: the current pair enters the read through u)
+ * Inputs are columns of the fp32 rows y (stride ldy): q, k [heads * dk], v, gate [heads * dv], low [rank]; q is scaled by
+ * q_scale.  decay = f(W2 act(low) + bias): DET_DECAY_SIGMOID: sigmoid(z)^(1/tau), act = identity; DET_DECAY_EXP:
+ * exp(-exp(z)), act = tanh.  out[row][head * dv + j] = o / sqrt(mean over dv of o^2 + eps) * norm[head * dv + j] *
+ * silu(gate), in the activation type.  `scratch` (det_f_recur_scratch_bytes) serves calls over several tokens of one
+ * sequence.  seq.one.s / table[].s hold S.                                                                             */
+#define DET_DECAY_SIGMOID 0
+#define DET_DECAY_EXP 1
+typedef struct {
+    int heads, dk, dv, rank;
+    int M;
+    int dtype;
+    const float* y;
+    int ldy;
+    int q_off, k_off, v_off, gate_off, low_off;
+    float q_scale;
+    int decay;
+    float tau;
+    const det_flinear* w2;    /* [heads * dk][rank] */
+    const float* bias;        /* [heads * dk] */
+    const float* u;           /* [heads * dk] or NULL */
+    const float* norm;        /* [heads * dv] */
+    float eps;
+    void* out;
+    int ldo;
+    void* scratch;
+    det_seq_ref seq;
+} det_frecur_op;
+void det_f_recur(const det_frecur_op* op, cudaStream_t st);
+size_t det_f_recur_scratch_bytes(int M, int heads, int dk, int dv);
+
+/* Latent attention.  A cache row is [c: kv_rank | zeros to a multiple of 8 | rotated key part: rot_dim | zeros], ld
+ * elements of the activation type (det_f_latent_ld).
+ * det_f_latent_prep: from the fp32 rows y, cq[row] = RMS norm of the q_rank columns at dq_off (weight dq_norm), the cache
+ * row of the token = RMS norm of the kv_rank columns at dkv_off (weight dkv_norm) and the rotation of the rot_dim columns
+ * behind them (pairs (2i, 2i+1), the first rot_dims of them; tables [position][rot_dims / 2]).
+ * det_f_latent_attn: q[row][heads * (dim + rot_dim)] fp32 (not yet rotated) attends the cached positions j with
+ * 0 <= i - j < window (window <= 0: all); per head softmax(scale * (q . W_uk c + q_rot . k_rot)) with exp(sink[head]) added
+ * to the denominator (sink NULL: none), values W_uv c; out[row][head * vdim + j] = value * sigmoid(gate), in the activation
+ * type.  wkv holds the rows of W_uk [heads * dim] followed by those of W_uv [heads * vdim].  max_pos bounds the positions.
+ * The caller guarantees cap >= min(window - 1 + M, positions in use).                                                  */
+typedef struct {
+    int heads, dim, rot_dim, rot_dims, vdim, q_rank, kv_rank;
+    int window;
+    float scale;
+    int cap;
+    int M;
+    int dtype;
+    const float* y;
+    int ldy;
+    int dq_off, dkv_off, gate_off;
+    const float* dq_norm;
+    const float* dkv_norm;
+    float eps;
+    const float* rope_cos;
+    const float* rope_sin;
+    void* cq;
+    int ldcq;
+    const float* q;
+    int ldq;
+    const det_flinear* wkv;
+    const float* sink;
+    void* out;
+    int ldo;
+    int max_pos;
+    void* scratch;
+    det_seq_ref seq;
+} det_flatent_op;
+int det_f_latent_ld(int kv_rank, int rot_dim);
+size_t det_f_latent_scratch_bytes(int M, int heads, int dim, int rot_dim, int vdim, int kv_rank, int window, int cap, int max_pos,
+                                  int dtype);
+void det_f_latent_prep(const det_flatent_op* op, cudaStream_t st);
+void det_f_latent_attn(const det_flatent_op* op, cudaStream_t st);
+
+/* Measurement switches of the floating-point ops (results agree up to rounding): bit 0 no norm in the GEMV's prologue, bit 1 no
+ * GEMV, bit 2 no split of K in the tensor-core GEMM, bit 3 no tensor-core attention.                                   */
+void det_debug_set_float(int flags);
+
 #ifdef __cplusplus
 }
 #endif

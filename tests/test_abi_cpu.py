@@ -75,7 +75,9 @@ def test_ctypes_mirror_has_the_layout_the_c_compiler_gives_the_header(libs, tmp_
         pytest.skip("needs gcc and the CUDA headers")
     pairs = {"det_qlinear": libs.QLinear, "det_attn_layer": libs.AttnLayer, "det_kv_cache": libs.KvCache,
              "det_gdn_layer": libs.GdnLayer, "det_gdn_state": libs.GdnState, "det_act_source": libs.ActSource,
-             "det_gemv_op": libs.GemvOp}
+             "det_gemv_op": libs.GemvOp, "det_flinear": libs.FLinear, "det_seq_slot": libs.SeqSlot,
+             "det_seq_ref": libs.SeqRef, "det_fnorm_op": libs.FNormOp, "det_fgemm_op": libs.FGemmOp,
+             "det_frecur_op": libs.FRecurOp, "det_flatent_op": libs.FLatentOp}
     lines = ['#include <stdio.h>', '#include <stddef.h>', '#include "det_b200.h"', "int main(void) {"]
     for cname, mirror in pairs.items():
         lines.append(f'  printf("{cname} %zu\\n", sizeof({cname}));')
