@@ -672,6 +672,140 @@ def run_serving(args, rank: int, world: int, local_rank: int):
     h.dh_batch_free(batch)
 
 
+def hybrid_config(width: int, ff: int, vocab: int, layers: int, window: int = 4096) -> dict:
+    """A hybrid decoder whose layers have the sizes of a real model: [gla, wkv, latent attention, gla] repeated."""
+    gla = {"type": "gla", "mixer": {"heads": width // 256, "dim": 128, "vdim": 256, "tau": 16.0}}
+    wkv = {"type": "wkv", "mixer": {"heads": width // 64, "dim": 64}}
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": width // 128, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": width * 3 // 10, "kv_rank": 512,
+                     "mask": {"size": window}, "rot": {"base": 10000.0, "dims": 64}, "scale": 192 ** -0.5}}
+    kinds = [gla, wkv, lat, gla]
+    return {"architecture": "Fazilorn", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [{**kinds[i % 4], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+def run_hybrid(args, rank: int, world: int, local_rank: int):
+    """The hybrid decoder (bfloat16, seeded random weights) beside the Qwen3.5-shaped quantized model of the same width,
+    feed-forward, vocabulary and depth: prefill, graph-replayed decode of one sequence, and a batched step.  One line; the
+    headline workload is another (`--workload decode`).  Reduced depth: the layers are those of a real model, not their number."""
+    import numpy as np
+    from det_b200 import capi
+    if world != 1:
+        raise RuntimeError("the hybrid workload runs on one GPU")
+    rt = C.CDLL("libcudart.so.12")
+    assert rt.cudaSetDevice(local_rank) == 0
+    h, d = capi.host(), capi.cuda()
+    bk = h.dh_cuda_backend_new(1, 1)
+    if not bk:
+        raise RuntimeError(h.dh_last_error().decode())
+    d.det_debug_set_float(args.float_flags)
+    K, W, layers = args.steps, args.warmup, args.layers or 8
+    ev = Events(d.det_cuda_stream())
+    sampler = ClockSampler(local_rank)
+    sampler.start()
+    windows = []
+    hbm, kind = _peaks()
+
+    def timed(fn, reps=1):
+        d.det_sync()
+        w0 = time.time()
+        a = ev.record()
+        for _ in range(reps):
+            fn()
+        b = ev.record()
+        ms = ev.ms(a, b) / reps
+        windows.append((w0, time.time()))
+        return ms
+
+    def measure(model, vocab, weight_bytes):
+        out = {}
+        P, chunk = args.prefill, args.chunk
+        ids = _prompt(h, P, vocab)
+        prefill = lambda: (_check(h.dh_model_reset(model), h), _check(h.dh_model_prefill(model, ids.ctypes.data, P), h))
+        prefill()
+        prefill()
+        prefill()
+        ms = timed(prefill)
+        out["prefill"] = {"tokens": P, "chunk": chunk, "ms": ms, "value": P / ms * 1e3, "unit": "tok/s"}
+        tok, rng = C.c_int32(0), C.c_uint64(0)
+        _check(h.dh_model_pick(model, 1, 1.0, 0, 1.0, C.byref(rng), C.byref(tok)), h)
+        dec = h.dh_graph_decoder_new(model)
+        if not dec:
+            raise RuntimeError(h.dh_last_error().decode())
+        buf = np.zeros(max(K, W), np.int32)
+        _check(h.dh_graph_decoder_enqueue(dec, tok.value, W, 1), h)
+        n = h.dh_graph_decoder_finish(dec, buf.ctypes.data, buf.size)
+        last = int(buf[n - 1])
+        rt.cudaProfilerStart()
+        ms = timed(lambda: _check(h.dh_graph_decoder_enqueue(dec, last, K, 1), h)) / K
+        rt.cudaProfilerStop()
+        h.dh_graph_decoder_finish(dec, buf.ctypes.data, buf.size)
+        h.dh_graph_decoder_free(dec)
+        out["decode"] = {"ms_per_token": ms, "value": 1e3 / ms, "unit": "tok/s", "context": P + W,
+                         "weight_gbs": weight_bytes / ms / 1e6, "frac_of_hbm": weight_bytes / ms / 1e6 / hbm}
+        # e2e of one token: token ids from the host, logits picked on the device, the id read back
+        one, t = np.array([last], np.int32), C.c_int32(0)
+
+        def eager():
+            _check(h.dh_model_forward(model, one.ctypes.data, 1), h)
+            _check(h.dh_model_pick(model, 1, 1.0, 0, 1.0, C.byref(rng), C.byref(t)), h)
+            one[0] = t.value
+        for _ in range(W):
+            eager()
+        ms = timed(eager, K)
+        out["e2e_decode"] = {"ms_per_token": ms, "value": 1e3 / ms, "unit": "tok/s", "h2d_bytes_per_step": 4, "d2h_bytes_per_step": 4}
+        if args.seqs > 1:
+            B = min(args.seqs, chunk)
+            ctxs = [int(x) for x in np.random.default_rng(SEED).integers(args.ctx_min, min(args.ctx_max, P) + 1, B)]
+            batch = h.dh_batch_new(model, B, max(ctxs) + K + W + 2)
+            if not batch:
+                raise RuntimeError(h.dh_last_error().decode())
+            for i, n in enumerate(ctxs):
+                _check(h.dh_batch_prefill(batch, i, ids.ctypes.data, n, 1, 1.0, 0, 1.0, 0), h)
+            _check(h.dh_batch_step(batch, W), h)
+            ms = timed(lambda: _check(h.dh_batch_step(batch, 1), h), K)
+            out["batch"] = {"sequences": B, "contexts": [min(ctxs), max(ctxs)], "ms_per_step": ms, "value": B / ms * 1e3, "unit": "tok/s"}
+            h.dh_batch_free(batch)
+        if d.det_last_error():
+            raise RuntimeError("a device-side wait reported an error")
+        return out
+
+    sizes = {}
+    ctx = args.prefill + 2 * (K + W) + 16
+    for name in args.sizes.split(","):
+        shape = SHAPES[name]
+        cfg = hybrid_config(shape["hidden"], shape["ffn"], shape["vocab"], layers)
+        res = {"width": shape["hidden"], "ff": shape["ffn"], "vocab": shape["vocab"], "layers": layers}
+        if "hybrid" in args.arms:
+            m = h.dh_hybrid_new_synth(bk, json.dumps(cfg).encode(), SEED, capi.DET_BF16, ctx, args.chunk)
+            if not m:
+                raise RuntimeError(h.dh_last_error().decode())
+            wb = h.dh_hybrid_weight_bytes(m)
+            res["hybrid"] = {"weight_bytes": wb, **measure(m, shape["vocab"], wb)}
+            h.dh_model_free(m)
+        if "qwen35" in args.arms:
+            m = h.dh_model_new_synth(bk, name.encode(), layers, SEED, ctx, args.chunk)
+            if not m:
+                raise RuntimeError(h.dh_last_error().decode())
+            head = shape["vocab"] * (shape["hidden"] + 4 + shape["hidden"] // 128 * 2) / 1e9
+            wb = int(((_weights_gb(name) - head) * layers / shape["layers"] + head) * 1e9)
+            res["qwen35"] = {"weight_bytes": wb, **measure(m, shape["vocab"], wb)}
+            h.dh_model_free(m)
+        sizes[name] = res
+    time.sleep(0.3)
+    sampler.stop()
+    last = sizes[args.sizes.split(",")[-1]]
+    main_arm = last.get("hybrid") or last["qwen35"]
+    print(json.dumps({
+        "metric": "hybrid decoder (Fazilorn) decode tok/s bs1, reduced depth", "value": main_arm["decode"]["value"], "unit": "tok/s",
+        "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": main_arm["decode"]["ms_per_token"], "higher_is_better": True,
+        "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"layers_built": layers, "pattern": "gla, wkv, latent_attention, gla", "prefill": args.prefill, "chunk": args.chunk,
+                   "l2": "weights streamed per token exceed the 126 MB L2", "hbm_peak_gbs": hbm, "peak_kind": kind,
+                   "float_flags": args.float_flags},
+        "sizes": sizes, "clocks": sampler.summary(windows)}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -688,8 +822,12 @@ def main():
     ap.add_argument("--layers", type=int, default=0,
                     help="build only the first L layers of the configuration (a small case for profiler captures; the "
                          "line says so and is not a result)")
-    ap.add_argument("--workload", default="decode", choices=["decode", "serving"],
-                    help="decode: the headline batch-1 token loop; serving: many sequences, one batched step per token")
+    ap.add_argument("--workload", default="decode", choices=["decode", "serving", "hybrid"],
+                    help="decode: the headline batch-1 token loop; serving: many sequences, one batched step per token; "
+                         "hybrid: the bfloat16 hybrid decoder beside the quantized model of equal size")
+    ap.add_argument("--sizes", default="4b,27b", help="hybrid: widths to run, comma separated names of the shapes")
+    ap.add_argument("--arms", default="hybrid,qwen35", help="hybrid: which of the two models to run")
+    ap.add_argument("--float-flags", type=int, default=0, help="hybrid: measurement switches (det_debug_set_float)")
     ap.add_argument("--seqs", type=int, default=32)
     ap.add_argument("--ctx-min", type=int, default=512)
     ap.add_argument("--ctx-max", type=int, default=8192)
@@ -727,7 +865,9 @@ def main():
         if world == 1:
             from det_b200 import capi
             capi.host().dh_use_cuda_synth_rows(1)   # the cpu_baseline leg builds its weights with the device generator
-        if args.workload == "serving":
+        if args.workload == "hybrid":
+            run_hybrid(args, rank, world, local_rank)
+        elif args.workload == "serving":
             run_serving(args, rank, world, local_rank)
         else:
             run_ours(args, rank, world, local_rank)

@@ -5,8 +5,9 @@
 // of K of both operands (128-byte rows, SWIZZLE_128B).  Persistent: a CTA walks its tiles, tokens fastest, with two TMEM
 // accumulators, so that the epilogue of one tile runs beside the loads and products of the next.  Warp 0 issues TMA, warp 1
 // the MMAs, the others drain TMEM and apply the epilogue (residual add, softcap, SwiGLU of interleaved gate / up rows).
-// A launch with few tiles splits K over several CTAs: partial sums go to the library's workspace and the CTA that arrives
-// last adds them in split order, so the result does not depend on the order of arrival.
+// When whole tiles would leave SMs idle in the last round, the stages of all tiles are dealt out evenly instead: a CTA may then
+// begin or end inside a tile.  Such a piece goes to the library's workspace, and the CTA that arrives last at the tile adds
+// its pieces in order of K, so the result does not depend on the order of arrival.
 #include "umma.cuh"
 #include "fops.cuh"
 #include <algorithm>
@@ -30,10 +31,11 @@ struct FtCfg {
 };
 
 struct FtPlan {
-    int tok_tiles, items, ksplit, kb;     // kb: stages over the whole of K
+    int tok_tiles, tiles, kb;             // kb: stages over the whole of K
+    int dealt;                            // stages are dealt out evenly (else whole tiles)
     int m_rows;                           // rows of one input group in the tensor map
-    float* part;
-    unsigned* counters;
+    float* part;                          // [CTA][2][TOK][FT_ROWS]: a piece that continues a tile, a piece that begins one
+    unsigned* counters;                   // one per CTA that begins a shared tile
 };
 
 __device__ __forceinline__ void umma_bf16(unsigned tmem_d, unsigned long long da, unsigned long long db, unsigned idesc,
@@ -46,20 +48,29 @@ __device__ __forceinline__ void umma_bf16(unsigned tmem_d, unsigned long long da
         : "memory");
 }
 
+// The run of stages of a CTA, [lo, hi) over all tiles: whole tiles, or an even share.
+__device__ __forceinline__ long long ft_bound(const FtPlan& p, int cta) {
+    if (!p.dealt) return (long long)cta * p.tiles / gridDim.x * p.kb;
+    return (long long)cta * p.tiles * p.kb / gridDim.x;
+}
+// The CTA whose run holds stage u.
+__device__ __forceinline__ int ft_owner(const FtPlan& p, long long u) {
+    int c = (int)(u * gridDim.x / ((long long)p.tiles * p.kb));
+    while (c + 1 < (int)gridDim.x && ft_bound(p, c + 1) <= u) c++;
+    while (c > 0 && ft_bound(p, c) > u) c--;
+    return c;
+}
 struct FtItem {
     TilePlace pl;
-    int wt, tt, ks, b0, nb;               // weight tile, token tile, split, first stage and number of stages
+    int tile, tt, b0, nb;                 // token tile; first stage and number of stages
 };
-__device__ __forceinline__ FtItem ft_item(const FgemmArgs& a, const FtPlan& p, int i) {
+__device__ __forceinline__ FtItem ft_item(const FgemmArgs& a, const FtPlan& p, long long u, long long hi) {
     FtItem it;
-    it.ks = i % p.ksplit;
-    const int tile = i / p.ksplit;
-    it.tt = tile % p.tok_tiles;
-    it.wt = tile / p.tok_tiles;
-    it.pl = place_tile<FT_ROWS>(a, it.wt);
-    const int per = (p.kb + p.ksplit - 1) / p.ksplit;
-    it.b0 = it.ks * per;
-    it.nb = max(0, min(p.kb, it.b0 + per) - it.b0);
+    it.tile = (int)(u / p.kb);
+    it.b0 = (int)(u % p.kb);
+    it.nb = (int)min((long long)(p.kb - it.b0), hi - u);
+    it.tt = it.tile % p.tok_tiles;
+    it.pl = place_tile<FT_ROWS>(a, it.tile / p.tok_tiles);
     return it;
 }
 
@@ -124,12 +135,13 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
     __syncthreads();
     tc_fence_after();
     const unsigned tmem = *tmem_slot;
+    const long long lo = ft_bound(p, blockIdx.x), hi = ft_bound(p, blockIdx.x + 1);
     bool ok = true;
 
     if (warp == 0) {
         if (lane == 0) {
             // the weight boxes of the first stages do not depend on the previous kernel
-            const FtItem first = ft_item(a, p, blockIdx.x);
+            const FtItem first = ft_item(a, p, lo, hi);
             const int lead = min(first.nb, STAGES);
             for (int l = 0; l < lead; l++) {
                 mbar_expect_tx(&full[l], Cfg::STAGE_BYTES);
@@ -137,8 +149,9 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
             }
             pdl_wait();
             unsigned c = 0;                          // stages issued so far
-            for (int i = blockIdx.x; i < p.items && ok; i += gridDim.x) {
-                const FtItem it = ft_item(a, p, i);
+            for (long long i = lo; i < hi && ok;) {
+                const FtItem it = ft_item(a, p, i, hi);
+                i += it.nb;
                 const int row = a.seg_in[it.pl.seg] * p.m_rows + it.tt * TOK;
                 for (int l = 0; l < it.nb; l++, c++) {
                     const int s = c % STAGES;
@@ -161,8 +174,9 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
     } else if (warp == 1) {
         if (lane == 0) {
             unsigned c = 0, t = 0;
-            for (int i = blockIdx.x; i < p.items && ok; i += gridDim.x, t++) {
-                const FtItem it = ft_item(a, p, i);
+            for (long long i = lo; i < hi && ok; t++) {
+                const FtItem it = ft_item(a, p, i, hi);
+                i += it.nb;
                 const unsigned b = t & 1u;
                 ok = mbar_wait(&tempty[b], ((t >> 1) & 1u) ^ 1u, wl);
                 if (!ok) break;
@@ -186,64 +200,64 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
         const int q = warp & 3, col0 = ((warp - 2) >> 2) * Cfg::EC, et = threadIdx.x - 64;
         pdl_wait();
         unsigned t = 0;
-        for (int i = blockIdx.x; i < p.items && ok; i += gridDim.x, t++) {
-            const FtItem it = ft_item(a, p, i);
+        constexpr size_t PIECE = (size_t)TOK * FT_ROWS;
+        for (long long i = lo; i < hi && ok; t++) {
+            const FtItem it = ft_item(a, p, i, hi);
+            i += it.nb;
             const unsigned b = t & 1u;
             ok = mbar_wait(&tfull[b], (t >> 1) & 1u, wl);
             if (!ok) break;
             tc_fence_after();
             const int n = it.pl.n0 + q * 32 + lane, m0 = it.tt * TOK + col0;
             const unsigned taddr = tmem + ((unsigned)(q * 32) << 16) + b * TOK + col0;
-            if (p.ksplit == 1) {
-                for (int c = 0; c < Cfg::EC; c += 32) {
-                    int r[32];
-                    tmem_ld(taddr + c, r);
-                    tmem_wait_ld();
-                    if (c + 32 >= Cfg::EC) {
-                        tc_fence_before();
-                        __syncwarp();
-                        if (lane == 0) mbar_arrive(&tempty[b]);
-                    }
-                    if (m0 + c < a.M) {
-#pragma unroll
-                        for (int j = 0; j < 32; j += 2)
-                            ft_emit2(a, it.pl, n, m0 + c + j, __int_as_float(r[j]), __int_as_float(r[j + 1]));
-                    }
-                }
-            } else {
-                // split K (TOK == 32, four epilogue warps, EC == 32): one partial tile per split
-                __shared__ unsigned last_cta;
-                const int tile = i / p.ksplit;
+            const bool whole = it.nb == p.kb;
+            float* mine = p.part + ((size_t)blockIdx.x * 2 + (it.b0 == 0 ? 1 : 0)) * PIECE + (size_t)col0 * FT_ROWS + q * 32 + lane;
+            for (int c = 0; c < Cfg::EC; c += 32) {
                 int r[32];
-                tmem_ld(taddr, r);
+                tmem_ld(taddr + c, r);
                 tmem_wait_ld();
-                tc_fence_before();
-                __syncwarp();
-                if (lane == 0) mbar_arrive(&tempty[b]);
-                float* mine = p.part + ((size_t)tile * p.ksplit + it.ks) * (FT_ROWS * 32) + q * 32 + lane;
+                if (c + 32 >= Cfg::EC) {
+                    tc_fence_before();
+                    __syncwarp();
+                    if (lane == 0) mbar_arrive(&tempty[b]);
+                }
+                if (m0 + c >= a.M) continue;
+                if (whole) {
 #pragma unroll
-                for (int j = 0; j < 32; j++) mine[j * FT_ROWS] = __int_as_float(r[j]);
+                    for (int j = 0; j < 32; j += 2)
+                        ft_emit2(a, it.pl, n, m0 + c + j, __int_as_float(r[j]), __int_as_float(r[j + 1]));
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 32; j++) mine[(size_t)(c + j) * FT_ROWS] = __int_as_float(r[j]);
+                }
+            }
+            if (whole) continue;
+            // a piece: the tile's CTAs meet at a counter; the last one adds the pieces
+            __shared__ unsigned last_cta;
+            const long long u0 = (long long)it.tile * p.kb;
+            const int first_cta = ft_owner(p, u0), end_cta = ft_owner(p, u0 + p.kb - 1);
+            __threadfence();
+            asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
+            if (et == 0) last_cta = atomicAdd(p.counters + first_cta, 1u) == (unsigned)(end_cta - first_cta);
+            asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
+            if (last_cta) {
                 __threadfence();
-                asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
-                if (et == 0) last_cta = atomicAdd(p.counters + tile, 1u) == (unsigned)p.ksplit - 1;
-                asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
-                if (last_cta) {
-                    __threadfence();
-                    const float* all = p.part + (size_t)tile * p.ksplit * (FT_ROWS * 32) + q * 32 + lane;
+                if (et == 0) p.counters[first_cta] = 0;
+                const float* all = p.part + (size_t)col0 * FT_ROWS + q * 32 + lane;
+                for (int c = 0; c < Cfg::EC && m0 + c < a.M; c += 32) {
                     float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; j++) v[j] = 0.0f;
-                    for (int s = 0; s < p.ksplit; s++)
+                    for (int s = first_cta; s <= end_cta; s++) {
+                        const float* piece = all + ((size_t)s * 2 + (s == first_cta ? 1 : 0)) * PIECE + (size_t)c * FT_ROWS;
 #pragma unroll
-                        for (int j = 0; j < 32; j++)
-                            if (m0 + j < a.M) v[j] += __ldcg(all + (size_t)s * (FT_ROWS * 32) + j * FT_ROWS);
-                    if (et == 0) p.counters[tile] = 0;
+                        for (int j = 0; j < 32; j++) v[j] += __ldcg(piece + (size_t)j * FT_ROWS);
+                    }
 #pragma unroll
-                    for (int j = 0; j < 32; j += 2)
-                        if (m0 + j < a.M) ft_emit2(a, it.pl, n, m0 + j, v[j], v[j + 1]);
+                    for (int j = 0; j < 32; j += 2) ft_emit2(a, it.pl, n, m0 + c + j, v[j], v[j + 1]);
                 }
-                asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");   // last_cta is read before it is written again
             }
+            asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");   // last_cta is read before it is written again
         }
         if (!ok && lane == 0) atomicExch(a.error_flag, DETB_ERR_WAIT_EXPIRED);
     }
@@ -275,20 +289,24 @@ static void launch_tok(FgemmArgs a, cudaStream_t q) {
     FtPlan p{};
     p.tok_tiles = (a.M + TOK - 1) / TOK;
     p.kb = (a.K + FT_KE - 1) / FT_KE;
-    p.ksplit = 1;
-    const int tiles = a.tile0[a.nseg] * p.tok_tiles, sms = sm_count();
-    if (TOK == 32 && !(float_flags() & 4)) {
+    p.tiles = a.tile0[a.nseg] * p.tok_tiles;
+    const int sms = sm_count();
+    int grid = std::min(p.tiles, sms);
+    if (!(float_flags() & 4)) {
+        // deal out stages when whole tiles keep less than 92 % of the SM-rounds busy, and a share is worth the hand-over
+        const long long units = (long long)p.tiles * p.kb;
+        const int rounds = (p.tiles + sms - 1) / sms, share = TOK == 32 ? 6 : 16;
+        const int want = (int)std::min<long long>(sms, units / share);
         size_t bytes = 0;
         int ncnt = 0;
         p.part = fsplit_workspace(&bytes);
         p.counters = fsplit_counters(&ncnt);
-        // fill the SMs, at least four stages of K per CTA
-        const int want = std::min({sms / std::max(tiles, 1), p.kb / 4, 16});
-        if (want > 1 && tiles <= ncnt && (size_t)tiles * want * FT_ROWS * 32 * sizeof(float) <= bytes) p.ksplit = want;
-        // every split owns at least one stage
-        while (p.ksplit > 1 && (p.ksplit - 1) * ((p.kb + p.ksplit - 1) / p.ksplit) >= p.kb) p.ksplit--;
+        if (p.tiles < 0.92 * rounds * sms && want >= grid && want <= ncnt &&
+            (size_t)want * 2 * TOK * FT_ROWS * sizeof(float) <= bytes) {
+            p.dealt = 1;
+            grid = want;
+        }
     }
-    p.items = tiles * p.ksplit;
     // input groups lie gstride elements apart; a map row is one row of the buffer
     DETB_REQUIRE(groups == 1 || a.gstride % a.ldx == 0, "input groups must be whole rows apart");
     p.m_rows = groups == 1 ? 0 : (int)(a.gstride / a.ldx);
@@ -301,7 +319,7 @@ static void launch_tok(FgemmArgs a, cudaStream_t q) {
         DETB_CUDA_OK(cudaFuncSetAttribute(k_fgemm_tc<TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM));
         configured = true;
     }
-    launch_pdl(k_fgemm_tc<TOK>, dim3(std::min(p.items, sms)), dim3(Cfg::THREADS), Cfg::SMEM, q, 1, map_w, map_x, a, p);
+    launch_pdl(k_fgemm_tc<TOK>, dim3(grid), dim3(Cfg::THREADS), Cfg::SMEM, q, 1, map_w, map_x, a, p);
 }
 
 void fgemm_tc_launch(FgemmArgs a, cudaStream_t q) {

@@ -6,10 +6,11 @@
 //     row is key and value at once.  k_latent_absorb: q W_uk per head; k_latent_scores: a warp per head walks a range of
 //     keys staged in shared memory, online softmax; k_latent_out merges the ranges, adds the sink, applies W_uv and the gate.
 //   expanded (a run of tokens with bfloat16 activations): keys and values of the cached rows are multiplied out by the
-//     tensor-core GEMM, then k_latent_flash computes 128 query rows of a head against 64-key tiles with bfloat16 MMAs.
+//     tensor-core GEMM, then k_latent_flash computes 64 query rows of a head against 64-key tiles with bfloat16 MMAs.
 #include "fops.cuh"
 #include <algorithm>
 #include <cmath>
+#include <type_traits>
 
 namespace detb {
 
@@ -75,37 +76,52 @@ __global__ void __launch_bounds__(256) k_latent_prep(const LatentArgs a) {
 
 // ------------------------------------------------------------------------------------------------------ absorbed form
 constexpr int AB_ROWS = 8;       // query rows per CTA
+constexpr int AB_COLS = 64;      // latent columns per CTA: two per lane; four warps share the head's dimensions
 __global__ void __launch_bounds__(128) k_latent_absorb(const LatentArgs a) {
-    extern __shared__ __align__(16) float qs[];      // [AB_ROWS][dim]
+    extern __shared__ __align__(16) float qs[];      // [AB_ROWS][dim], then the warps' partial sums [4][AB_ROWS][AB_COLS]
     const int h = blockIdx.x, r0 = blockIdx.z * AB_ROWS, nr = min(AB_ROWS, a.M - r0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    float* sums = qs + AB_ROWS * a.dim;
     pdl_trigger();
     pdl_wait();
     const int hd = a.dim + a.rot_dim;
-    for (int i = threadIdx.x; i < AB_ROWS * a.dim; i += 128) {
+    for (int i = threadIdx.x; i < nr * a.dim; i += 128) {
         const int r = i / a.dim, d = i % a.dim;
-        qs[i] = r < nr ? a.q[(size_t)(r0 + r) * a.ldq + h * hd + d] * a.scale : 0.0f;
+        qs[i] = a.q[(size_t)(r0 + r) * a.ldq + h * hd + d] * a.scale;
     }
     __syncthreads();
-    const int c = blockIdx.y * 256 + threadIdx.x * 2;
-    if (c < a.rp) {
-        float acc[AB_ROWS][2];
+    const int c = blockIdx.y * AB_COLS + lane * 2;
+    const bf16* w = a.wkv + (size_t)h * a.dim * a.ldw + min(c, a.rp - 2);      // rows padded with zeros to a multiple of 8
+    auto run = [&](auto rows) {
+        constexpr int R = decltype(rows)::value;
+        float acc[R][2];
 #pragma unroll
-        for (int r = 0; r < AB_ROWS; r++) acc[r][0] = acc[r][1] = 0.0f;
-        const bf16* w = a.wkv + (size_t)h * a.dim * a.ldw + c;      // rows padded with zeros to a multiple of 8
-#pragma unroll 8
-        for (int d = 0; d < a.dim; d++) {
-            const unsigned b = *reinterpret_cast<const unsigned*>(w + (size_t)d * a.ldw);
+        for (int r = 0; r < R; r++) acc[r][0] = acc[r][1] = 0.0f;
+#pragma unroll 16
+        for (int d = warp; d < a.dim; d += 4) {
+            const unsigned b = __ldg(reinterpret_cast<const unsigned*>(w + (size_t)d * a.ldw));
             const float w0 = bf_lo(b), w1 = bf_hi(b);
 #pragma unroll
-            for (int r = 0; r < AB_ROWS; r++) {
+            for (int r = 0; r < R; r++) {
                 const float q = qs[r * a.dim + d];
                 acc[r][0] = fmaf(q, w0, acc[r][0]);
                 acc[r][1] = fmaf(q, w1, acc[r][1]);
             }
         }
 #pragma unroll
-        for (int r = 0; r < AB_ROWS; r++)
-            if (r < nr) *reinterpret_cast<float2*>(a.qa + ((size_t)(r0 + r) * a.heads + h) * a.ld + c) = make_float2(acc[r][0], acc[r][1]);
+        for (int r = 0; r < R; r++) *reinterpret_cast<float2*>(sums + (warp * AB_ROWS + r) * AB_COLS + lane * 2) = make_float2(acc[r][0], acc[r][1]);
+    };
+    if (nr == 1) run(std::integral_constant<int, 1>{});
+    else run(std::integral_constant<int, AB_ROWS>{});
+    __syncthreads();
+    for (int i = threadIdx.x; i < nr * AB_COLS; i += 128) {
+        const int r = i / AB_COLS, cc = i % AB_COLS, col = blockIdx.y * AB_COLS + cc;
+        if (col < a.rp) {
+            float v = 0.0f;
+#pragma unroll
+            for (int k = 0; k < 4; k++) v += sums[(k * AB_ROWS + r) * AB_COLS + cc];
+            a.qa[((size_t)(r0 + r) * a.heads + h) * a.ld + col] = v;
+        }
     }
     if (blockIdx.y == 0)
         for (int i = threadIdx.x; i < nr * (a.ld - a.rp); i += 128) {
@@ -138,8 +154,8 @@ __global__ void __launch_bounds__(LS_WARPS * 32) k_latent_scores(const LatentArg
     const int row = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y * LS_WARPS + warp;
     pdl_trigger();
-    // columns past the row's end stay zero
-    for (int i = threadIdx.x; i < 2 * LS_KEYS * LDT; i += LS_WARPS * 32) put(tile + i, 0.0f);
+    // columns past a row's end stay zero; so do rows before their first use
+    for (int i = threadIdx.x; i < 2 * LS_KEYS * LDT / VEC; i += LS_WARPS * 32) reinterpret_cast<uint4*>(tile)[i] = make_uint4(0, 0, 0, 0);
     pdl_wait();
     const int pos = position_of(a.seq, row);
     const int lo = first_key(pos, a.window) + blockIdx.x * a.per_split, hi = min(pos + 1, lo + a.per_split);
@@ -154,13 +170,14 @@ __global__ void __launch_bounds__(LS_WARPS * 32) k_latent_scores(const LatentArg
     float m = -INFINITY, l = 0.0f;
     const int vecs = a.ld / VEC;
     auto fetch = [&](int k0, int buf) {
-        for (int i = threadIdx.x; i < LS_KEYS * vecs; i += LS_WARPS * 32) {
-            const int k = i / vecs, v = i % vecs;
-            if (k0 + k < hi) {
-                const T* src = cache + (size_t)((k0 + k) % a.cap) * a.ld + v * VEC;
-                const unsigned dst = smem_addr(tile + ((size_t)buf * LS_KEYS + k) * LDT + v * VEC);
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-            }
+        const int slot0 = k0 % a.cap;
+        for (int k = warp; k < LS_KEYS && k0 + k < hi; k += LS_WARPS) {      // a warp copies a row
+            int slot = slot0 + k;
+            while (slot >= a.cap) slot -= a.cap;
+            const T* src = cache + (size_t)slot * a.ld;
+            const T* dst = tile + ((size_t)buf * LS_KEYS + k) * LDT;
+            for (int v = lane; v < vecs; v += 32)
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst + v * VEC)), "l"(src + v * VEC) : "memory");
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -244,7 +261,7 @@ __global__ void __launch_bounds__(LS_WARPS * 32) k_latent_scores(const LatentArg
     }
 }
 
-constexpr int LO_V = 64;      // value dimensions per CTA
+constexpr int LO_V = 32;      // value dimensions per CTA
 template <class T>
 __global__ void __launch_bounds__(256) k_latent_out(const LatentArgs a) {
     extern __shared__ __align__(16) float osm[];
@@ -274,9 +291,10 @@ __global__ void __launch_bounds__(256) k_latent_out(const LatentArgs a) {
     const float inv = total;
     for (int r = threadIdx.x; r < ((a.kv_rank + 7) & ~7); r += 256) {
         float o = 0.0f;
-        if (r < a.kv_rank)
-            for (int s = 0; s < a.splits; s++)
-                if (fac[s] > 0.0f) o = fmaf(fac[s], part[(size_t)s * pr + 2 + r], o);
+        if (r < a.kv_rank) {
+#pragma unroll 8
+            for (int s = 0; s < a.splits; s++) o = fmaf(fac[s], part[(size_t)s * pr + 2 + r], o);
+        }
         ol[r] = o * inv;
     }
     __syncthreads();
@@ -304,7 +322,7 @@ __global__ void __launch_bounds__(256) k_latent_out(const LatentArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------------------ expanded form
-constexpr int FL_ROWS = 128, FL_KEYS = 64, FL_WARPS = 8;
+constexpr int FL_ROWS = 64, FL_KEYS = 64, FL_WARPS = 4;
 
 __device__ __forceinline__ void ldsm4(unsigned addr, unsigned (&r)[4]) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -320,13 +338,13 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const unsigned (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// One head x 128 query rows; DV = value dimensions rounded up to a multiple of 64.
+// One head x 64 query rows; DV = value dimensions rounded up to a multiple of 64.
 template <int DV>
-__global__ void __launch_bounds__(FL_WARPS * 32, 1) k_latent_flash(const LatentArgs a) {
+__global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentArgs a) {
     extern __shared__ __align__(16) uint8_t fsm[];
     const int hd = a.dim + a.rot_dim, dqp = (hd + 15) & ~15, ldk = dqp + 8;
     constexpr int LDV = DV + 8;
-    bf16* Q = reinterpret_cast<bf16*>(fsm);                       // [128][ldk]
+    bf16* Q = reinterpret_cast<bf16*>(fsm);                       // [64][ldk]
     bf16* Kt = Q + FL_ROWS * ldk;                                  // [2][64][ldk]
     bf16* Vt = Kt + 2 * FL_KEYS * ldk;                             // [2][64][LDV]
     const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -350,23 +368,45 @@ __global__ void __launch_bounds__(FL_WARPS * 32, 1) k_latent_flash(const LatentA
     }
     const bf16* cache = static_cast<const bf16*>(a.seq.one.cache);
     const int kvec = a.dim / 8, rvec = a.rot_dim / 8, vvec = a.vdim / 8, tvec = kvec + rvec + vvec;
+    // a warp copies whole key rows; which pieces of a row a lane takes does not depend on the row
+    constexpr int PIECES = 3;
+    const bf16* piece[PIECES];
+    size_t step[PIECES];
+    bf16* to[PIECES];
+    int ldt[PIECES];
+#pragma unroll
+    for (int j = 0; j < PIECES; j++) {
+        const int v = lane + j * 32;
+        piece[j] = nullptr;
+        step[j] = 0;
+        to[j] = Kt;
+        ldt[j] = ldk;
+        if (v < kvec) {
+            piece[j] = a.kv + h * a.dim + v * 8;
+            step[j] = a.ldkv;
+            to[j] = Kt + v * 8;
+        } else if (v < kvec + rvec) {
+            piece[j] = cache + a.rp + (v - kvec) * 8;
+            step[j] = a.ld;
+            to[j] = Kt + v * 8;
+        } else if (v < tvec) {
+            piece[j] = a.kv + a.heads * a.dim + h * a.vdim + (v - kvec - rvec) * 8;
+            step[j] = a.ldkv;
+            to[j] = Vt + (v - kvec - rvec) * 8;
+            ldt[j] = LDV;
+        }
+    }
     auto fetch = [&](int k0, int buf) {
-        for (int i = threadIdx.x; i < FL_KEYS * tvec; i += NT) {
-            const int k = i / tvec, v = i % tvec, j = min(k0 + k, p_last);     // past the last key: a copy, masked below
-            const size_t slot = (size_t)(j % a.cap);
-            const bf16* src;
-            bf16* dst;
-            if (v < kvec) {
-                src = a.kv + slot * a.ldkv + h * a.dim + v * 8;
-                dst = Kt + ((size_t)buf * FL_KEYS + k) * ldk + v * 8;
-            } else if (v < kvec + rvec) {
-                src = cache + slot * a.ld + a.rp + (v - kvec) * 8;
-                dst = Kt + ((size_t)buf * FL_KEYS + k) * ldk + v * 8;
-            } else {
-                src = a.kv + slot * a.ldkv + a.heads * a.dim + h * a.vdim + (v - kvec - rvec) * 8;
-                dst = Vt + ((size_t)buf * FL_KEYS + k) * LDV + (v - kvec - rvec) * 8;
-            }
-            asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
+        const int slot0 = k0 % a.cap;
+        for (int k = warp; k < FL_KEYS; k += FL_WARPS) {
+            int slot = slot0 + min(k, p_last - k0);               // past the last key: a copy of it, masked below
+            while (slot >= a.cap) slot -= a.cap;
+#pragma unroll
+            for (int j = 0; j < PIECES; j++)
+                if (piece[j])
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(to[j] + (buf * FL_KEYS + k) * ldt[j])),
+                                 "l"(piece[j] + (size_t)slot * step[j])
+                                 : "memory");
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -499,7 +539,7 @@ static size_t flash_smem(int hd, int dv) {
 // Runs of at least 32 tokens of one sequence with bfloat16 activations and head sizes in whole 16-byte pieces.
 static bool takes_flash(int M, bool one_seq, int dtype, int heads, int dim, int rot_dim, int vdim) {
     return one_seq && dtype == DET_BF16 && M >= 32 && !(float_flags() & 8) && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 &&
-           vdim <= 256 && (heads * vdim) % 2 == 0 && flash_smem(dim + rot_dim, (vdim + 63) / 64 * 64) <= 220 * 1024;
+           vdim <= 256 && dim + rot_dim + vdim <= 768 && flash_smem(dim + rot_dim, (vdim + 63) / 64 * 64) <= 220 * 1024;
 }
 static int latent_rp(int kv_rank) { return round8(kv_rank); }
 
@@ -631,8 +671,10 @@ void det_f_latent_attn(const det_flatent_op* op, cudaStream_t st) {
     plan_splits(op->M, op->heads, op->window, op->max_pos, sm_count(), &a.splits, &a.per_split);
     a.qa = static_cast<float*>(op->scratch);
     a.part = a.qa + (size_t)op->M * op->heads * a.ld;
-    launch_pdl(k_latent_absorb, dim3(op->heads, (a.rp + 255) / 256, (op->M + AB_ROWS - 1) / AB_ROWS), dim3(128),
-               (size_t)AB_ROWS * op->dim * sizeof(float), q, 1, a);
+    const size_t absorb_smem = ((size_t)AB_ROWS * op->dim + 4 * AB_ROWS * AB_COLS) * sizeof(float);
+    DETB_REQUIRE(absorb_smem <= 48 * 1024, "latent attention: the head is too large");
+    launch_pdl(k_latent_absorb, dim3(op->heads, (a.rp + AB_COLS - 1) / AB_COLS, (op->M + AB_ROWS - 1) / AB_ROWS), dim3(128), absorb_smem,
+               q, 1, a);
     if (op->dtype == DET_BF16) scores<bf16>(a, q);
     else scores<float>(a, q);
     const size_t smem = ((size_t)round8(op->kv_rank) + a.splits) * sizeof(float);

@@ -31,7 +31,7 @@ struct Runtime {
     size_t attn_ws_bytes = 0;
     bool attn_ws_owned = false;
 };
-constexpr size_t FSPLIT_BYTES = 8u << 20;
+constexpr size_t FSPLIT_BYTES = 40u << 20;
 constexpr int FSPLIT_TILES = 512;
 Runtime* g_rt = nullptr;
 std::once_flag g_once;

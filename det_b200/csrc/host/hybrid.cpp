@@ -317,10 +317,11 @@ std::unique_ptr<HybridModel> HybridModel::load(const HybridConfig& cfg, TensorSo
     m.max_batch = max_batch;
     const bool synthetic = dynamic_cast<SynthSource*>(&src) != nullptr;
     const size_t W = cfg.width;
-    {
+    m.embed_ = bk->alloc<uint16_t>(cfg.vocab * W);
+    if (!src.on_device("embed", cfg.vocab, W, m.embed_.ptr())) {
         std::vector<uint16_t> e(cfg.vocab * W);
         src.matrix("embed", cfg.vocab, W, e.data());
-        m.embed_ = bk->upload(e);
+        bk->write(m.embed_, 0, e.data(), e.size());
         bk->sync();
     }
     m.weights_.resize(cfg.layers.size());
@@ -357,7 +358,7 @@ std::unique_ptr<HybridModel> HybridModel::load(const HybridConfig& cfg, TensorSo
     for (size_t i = 0; i < cfg.layers.size(); i++) {
         const HybridWeights& w = *m.weights_[i];
         const MixerSpec& x = cfg.layers[i].mixer;
-        ldy = std::max(ldy, w.plain);
+        ldy = std::max(ldy, round8(w.plain));
         cat = std::max(cat, w.out.ld);
         if (x.kind == MixerKind::Wkv) groups = 6;
         if (x.kind == MixerKind::Latent) {
@@ -482,7 +483,7 @@ void HybridModel::run_in(const LayerSpec& l, const HybridWeights& w, size_t t, c
         if (l.ff) segment(w.in.n, 0);
     }
     g.y = y_.ptr();
-    g.ldy = (int)w.plain;
+    g.ldy = (int)round8(w.plain);
     g.h = cat_.ptr() + w.out_ff * dtype_bytes(dtype);
     g.ldh = (int)w.out.ld;
     backend->f_gemm(g);
@@ -500,7 +501,7 @@ void HybridModel::mixer_recurrent(const LayerSpec& l, const HybridWeights& w, si
     r.M = (int)t;
     r.dtype = (int)dtype;
     r.y = y_.ptr();
-    r.ldy = (int)w.plain;
+    r.ldy = (int)round8(w.plain);
     r.q_off = (int)w.off[0];
     r.k_off = (int)w.off[1];
     r.v_off = (int)w.off[2];
@@ -538,7 +539,7 @@ void HybridModel::mixer_latent(const LayerSpec& l, const HybridWeights& w, size_
     a.M = (int)t;
     a.dtype = (int)dtype;
     a.y = y_.ptr();
-    a.ldy = (int)w.plain;
+    a.ldy = (int)round8(w.plain);
     a.dq_off = (int)w.off[0];
     a.dkv_off = (int)w.off[1];
     a.gate_off = (int)w.off[2];
