@@ -6,6 +6,9 @@ kernels that a profiler capture needs (a few hundred MB on the device, a handful
     python bench_kernel.py umma_peak                        # int8 tcgen05.mma issue rate with resident operands
     python bench_kernel.py stream_peak                      # HBM read rate with nothing to compute: plain loads, GEMV rings
     python bench_kernel.py attn [n_h n_kv M pos0 [tc]]      # prefill attention, default 24 4 512 1536, tensor path on
+    python bench_kernel.py fgemm [N K M]                    # bfloat16 product, default 5120 22528 512 (1 .. 4 rows: the GEMV)
+    python bench_kernel.py recur [gla|wkv heads dk dv M]    # linear recurrence, default gla 20 128 256 512
+    python bench_kernel.py latent [heads dim rot vdim kv_rank M pos0 window]   # default 40 128 64 128 512 512 1536 4096
 
 attn: one det_attention call of M tokens behind pos0 cached positions (head_dim 256, random cache contents); tc = 0
 keeps it on the CUDA-core kernels; 2 warm-up calls, then 5 timed ones.
@@ -117,6 +120,101 @@ def attn(argv):
     d.det_sync()
 
 
+def _rand(d, rng, shape, scale=1.0, bf16=False):
+    a = (rng.standard_normal(shape) * scale).astype(np.float32)
+    if bf16:
+        b = a.view(np.uint32)
+        a = ((b + 0x7FFF + ((b >> 16) & 1)) >> 16).astype(np.uint16)
+    p = d.det_malloc(a.nbytes)
+    d.det_memcpy(p, a.ctypes.data, a.nbytes, None)
+    d.det_sync()
+    return p
+
+
+def _time(ev, fn, reps=10):
+    for _ in range(3):
+        fn()
+    a = ev.record()
+    for _ in range(reps):
+        fn()
+    b = ev.record()
+    return ev.ms(a, b) / reps * 1e3
+
+
+def _flinear(d, rng, n, k, tiled=True):
+    ld = (k + 7) // 8 * 8
+    w = d.det_malloc(n * ld * 2)
+    d.det_synth_bf16(7, n + k, n * ld, w, None)
+    lin = capi.FLinear(w, n, k, ld, None)
+    if tiled:
+        ends = (C.c_int * 1)(n)
+        lin.wt = d.det_malloc(d.det_f_linear_tile_bytes(k, 1, ends))
+        d.det_f_linear_tile(C.byref(lin), 1, ends, lin.wt, None)
+    return lin
+
+
+def fgemm(argv):
+    n, k, m = map(int, argv[1:4]) if len(argv) >= 4 else (5120, 22528, 512)
+    d, rng = capi.cuda(), np.random.default_rng(1)
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+    copies = max(1, min(6, int(400e6 // (n * k * 2)) + 1))       # more than the L2 holds
+    lins = [_flinear(d, rng, n, k, tiled=m > 4) for _ in range(copies)]
+    x, y = _rand(d, rng, (m, k), bf16=True), d.det_malloc(m * n * 4)
+    ops = [capi.FGemmOp(lin=C.pointer(lin), dtype=capi.DET_BF16, x=x, ldx=k, nseg=1, seg_end=(C.c_int * 8)(n), glu_from=n, M=m, y=y, ldy=n)
+           for lin in lins]
+    turn = [0]
+
+    def call():
+        d.det_f_gemm(C.byref(ops[turn[0] % copies]), None)
+        turn[0] += 1
+
+    us = _time(ev, call, 12)
+    print(f"det_f_gemm N={n} K={k} M={m}: {us:.1f} us/launch, {2 * m * n * k / us / 1e6:.0f} TFLOP/s, {n * k * 2 / us / 1e3:.0f} GB/s of "
+          f"weights; device error word {d.det_last_error()}")
+
+
+def recur(argv):
+    kind, heads, dk, dv, m = (argv[1], *map(int, argv[2:6])) if len(argv) >= 6 else ("gla", 20, 128, 256, 512)
+    d, rng, rank = capi.cuda(), np.random.default_rng(1), 64
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+    qk, vo = heads * dk, heads * dv
+    ld = 2 * qk + 2 * vo + rank
+    lin = _flinear(d, rng, qk, rank, tiled=False)
+    op = capi.FRecurOp(heads=heads, dk=dk, dv=dv, rank=rank, M=m, dtype=capi.DET_BF16, y=_rand(d, rng, (m, ld)), ldy=ld, q_off=0, k_off=qk,
+                       v_off=2 * qk, gate_off=2 * qk + vo, low_off=2 * qk + 2 * vo, q_scale=dk ** -0.5, tau=16.0,
+                       decay=capi.DET_DECAY_SIGMOID if kind == "gla" else capi.DET_DECAY_EXP, w2=C.pointer(lin), bias=_rand(d, rng, qk),
+                       u=_rand(d, rng, qk) if kind == "wkv" else None, norm=_rand(d, rng, vo), eps=1e-5, out=d.det_malloc(m * vo * 2), ldo=vo,
+                       scratch=d.det_malloc(d.det_f_recur_scratch_bytes(m, heads, dk, dv)),
+                       seq=capi.SeqRef(one=capi.SeqSlot(s=d.det_malloc(heads * dk * dv * 4))))
+    us = _time(ev, lambda: d.det_f_recur(C.byref(op), None))
+    print(f"det_f_recur {kind} heads={heads} dk={dk} dv={dv} M={m}: {us:.1f} us/call, {3 * heads * dk * dv * m / us / 1e6:.2f} TFMA/s; "
+          f"device error word {d.det_last_error()}")
+
+
+def latent(argv):
+    h, dim, rot, vdim, r, m, pos0, window = map(int, argv[1:9]) if len(argv) >= 9 else (40, 128, 64, 128, 512, 512, 1536, 4096)
+    d, rng, q_rank = capi.cuda(), np.random.default_rng(1), 1536
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+    cap = min(window - 1 + m, pos0 + m) if window else pos0 + m
+    ld, ldy = d.det_f_latent_ld(r, rot), q_rank + r + rot + h * vdim
+    lin = _flinear(d, rng, h * (dim + vdim), r)
+    op = capi.FLatentOp(heads=h, dim=dim, rot_dim=rot, rot_dims=rot, vdim=vdim, q_rank=q_rank, kv_rank=r, window=window, scale=(dim + rot) ** -0.5,
+                        cap=cap, M=m, dtype=capi.DET_BF16, y=_rand(d, rng, (m, ldy)), ldy=ldy, dq_off=0, dkv_off=q_rank, gate_off=q_rank + r + rot,
+                        dq_norm=_rand(d, rng, q_rank), dkv_norm=_rand(d, rng, r), eps=1e-5, rope_cos=_rand(d, rng, ((pos0 + m), max(1, rot // 2))),
+                        rope_sin=_rand(d, rng, ((pos0 + m), max(1, rot // 2))), cq=d.det_malloc(m * q_rank * 2), ldcq=q_rank,
+                        q=_rand(d, rng, (m, h * (dim + rot))), ldq=h * (dim + rot), wkv=C.pointer(lin), sink=_rand(d, rng, h),
+                        out=d.det_malloc(m * h * vdim * 2), ldo=h * vdim, max_pos=pos0 + m - 1,
+                        scratch=d.det_malloc(d.det_f_latent_scratch_bytes(m, h, dim, rot, vdim, r, window, cap, pos0 + m - 1, capi.DET_BF16)),
+                        seq=capi.SeqRef(one=capi.SeqSlot(cache=_rand(d, rng, (cap, ld), bf16=True)), pos0=pos0))
+    us = _time(ev, lambda: d.det_f_latent_attn(C.byref(op), None))
+    keys = sum(min(window or 1 << 30, pos0 + i + 1) for i in range(m))
+    print(f"det_f_latent_attn heads={h} dim={dim}+{rot} vdim={vdim} kv_rank={r} M={m} pos0={pos0} window={window}: {us:.1f} us/call, "
+          f"{2 * h * keys * (dim + rot + vdim) / us / 1e6:.1f} TFLOP/s (expanded form); device error word {d.det_last_error()}")
+
+
 def main(argv):
     kind = argv[0] if argv else "gemv"
     if kind == "umma_peak":
@@ -154,6 +252,8 @@ def main(argv):
         return
     if kind == "attn":
         return attn(argv)
+    if kind in ("fgemm", "recur", "latent"):
+        return {"fgemm": fgemm, "recur": recur, "latent": latent}[kind](argv)
     if kind not in ("gemv", "gemm_tc"):
         raise SystemExit(__doc__)
     n, k, bits, m = (17408, 5120, 6, 1 if kind == "gemv" else 512)

@@ -58,7 +58,7 @@ class GemvOp(C.Structure):
 
 class FLinear(C.Structure):
     """det_flinear (include/det_b200.h, Part 3)."""
-    _fields_ = [("w", c_void_p), ("N", c_int), ("K", c_int), ("ld", c_int)]
+    _fields_ = [("w", c_void_p), ("N", c_int), ("K", c_int), ("ld", c_int), ("wt", c_void_p)]
 
 
 class SeqSlot(C.Structure):
@@ -185,6 +185,8 @@ CUDA_ABI = {
     "det_embed_table": (None, [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]),
     "det_f_norm": (None, [C.POINTER(FNormOp), c_void_p]),
     "det_f_gemm": (None, [C.POINTER(FGemmOp), c_void_p]),
+    "det_f_linear_tile_bytes": (c_size_t, [c_int, c_int, C.POINTER(c_int)]),
+    "det_f_linear_tile": (None, [C.POINTER(FLinear), c_int, C.POINTER(c_int), c_void_p, c_void_p]),
     "det_f_recur": (None, [C.POINTER(FRecurOp), c_void_p]),
     "det_f_recur_scratch_bytes": (c_size_t, [c_int, c_int, c_int, c_int]),
     "det_f_latent_ld": (c_int, [c_int, c_int]),

@@ -137,6 +137,7 @@ extern "C" void det_f_gemm(const det_fgemm_op* op, cudaStream_t st) {
     DETB_REQUIRE(op->nseg >= 1 && op->nseg <= 8 && op->seg_end[op->nseg - 1] == l.N, "linear: bad segments");
     FgemmArgs a{};
     a.w = static_cast<const bf16*>(l.w);
+    a.wt = static_cast<const bf16*>(l.wt);
     a.N = l.N; a.K = l.K; a.ldw = l.ld;
     a.x = op->x; a.ldx = op->ldx; a.gstride = op->group_stride;
     a.nseg = op->nseg;

@@ -31,10 +31,11 @@ struct FtCfg {
 };
 
 struct FtPlan {
-    int tok_tiles, tiles, kb;             // kb: stages over the whole of K
+    int tok_tiles, wtiles, kb;            // token tiles, weight tiles, stages over the whole of K
+    int tiled;                            // weights come from the tile-major copy
     int dealt;                            // stages are dealt out evenly (else whole tiles)
     int m_rows;                           // rows of one input group in the tensor map
-    float* part;                          // [CTA][2][TOK][FT_ROWS]: a piece that continues a tile, a piece that begins one
+    float* part;                          // [CTA][2][TOK][FT_ROWS]: the piece that continues a tile, the piece that begins one
     unsigned* counters;                   // one per CTA that begins a shared tile
 };
 
@@ -48,29 +49,59 @@ __device__ __forceinline__ void umma_bf16(unsigned tmem_d, unsigned long long da
         : "memory");
 }
 
-// The run of stages of a CTA, [lo, hi) over all tiles: whole tiles, or an even share.
-__device__ __forceinline__ long long ft_bound(const FtPlan& p, int cta) {
-    if (!p.dealt) return (long long)cta * p.tiles / gridDim.x * p.kb;
-    return (long long)cta * p.tiles * p.kb / gridDim.x;
-}
-// The CTA whose run holds stage u.
-__device__ __forceinline__ int ft_owner(const FtPlan& p, long long u) {
-    int c = (int)(u * gridDim.x / ((long long)p.tiles * p.kb));
-    while (c + 1 < (int)gridDim.x && ft_bound(p, c + 1) <= u) c++;
-    while (c > 0 && ft_bound(p, c) > u) c--;
-    return c;
-}
+// The pieces of a launch a CTA works on, one after the other.  Whole tiles are dealt round robin, tokens fastest.  Stages are
+// dealt per token tile: CTA c belongs to token tile c % tok_tiles, and the CTAs of a token tile share its (weight tile, stage)
+// sequence evenly, so that CTAs which read the same weights run side by side.
 struct FtItem {
     TilePlace pl;
-    int tile, tt, b0, nb;                 // token tile; first stage and number of stages
+    int wt, tt, b0, nb;                   // weight tile, token tile, first stage and number of stages
 };
-__device__ __forceinline__ FtItem ft_item(const FgemmArgs& a, const FtPlan& p, long long u, long long hi) {
+struct FtWalk {
+    long long u, hi;                      // dealt: stage positions; else tile numbers
+    int ctas, rank;                       // dealt: CTAs of this token tile and this one's place among them
+};
+__device__ __forceinline__ long long ft_bound(const FtPlan& p, const FtWalk& w, int rank) {
+    return (long long)rank * p.wtiles * p.kb / w.ctas;
+}
+__device__ __forceinline__ FtWalk ft_walk(const FtPlan& p) {
+    FtWalk w;
+    w.ctas = w.rank = 0;
+    if (!p.dealt) {
+        w.u = blockIdx.x;
+        w.hi = (long long)p.wtiles * p.tok_tiles;
+        return w;
+    }
+    const int tt = blockIdx.x % p.tok_tiles;
+    w.rank = blockIdx.x / p.tok_tiles;
+    w.ctas = (gridDim.x - tt + p.tok_tiles - 1) / p.tok_tiles;
+    w.u = ft_bound(p, w, w.rank);
+    w.hi = ft_bound(p, w, w.rank + 1);
+    return w;
+}
+// The rank whose run holds stage u.
+__device__ __forceinline__ int ft_owner(const FtPlan& p, const FtWalk& w, long long u) {
+    int c = (int)(u * w.ctas / ((long long)p.wtiles * p.kb));
+    while (c + 1 < w.ctas && ft_bound(p, w, c + 1) <= u) c++;
+    while (c > 0 && ft_bound(p, w, c) > u) c--;
+    return c;
+}
+__device__ __forceinline__ bool ft_more(const FtWalk& w) { return w.u < w.hi; }
+__device__ __forceinline__ FtItem ft_next(const FgemmArgs& a, const FtPlan& p, FtWalk& w) {
     FtItem it;
-    it.tile = (int)(u / p.kb);
-    it.b0 = (int)(u % p.kb);
-    it.nb = (int)min((long long)(p.kb - it.b0), hi - u);
-    it.tt = it.tile % p.tok_tiles;
-    it.pl = place_tile<FT_ROWS>(a, it.tile / p.tok_tiles);
+    if (p.dealt) {
+        it.wt = (int)(w.u / p.kb);
+        it.tt = blockIdx.x % p.tok_tiles;
+        it.b0 = (int)(w.u % p.kb);
+        it.nb = (int)min((long long)(p.kb - it.b0), w.hi - w.u);
+        w.u += it.nb;
+    } else {
+        it.wt = (int)(w.u / p.tok_tiles);
+        it.tt = (int)(w.u % p.tok_tiles);
+        it.b0 = 0;
+        it.nb = p.kb;
+        w.u += gridDim.x;
+    }
+    it.pl = place_tile<FT_ROWS>(a, it.wt);
     return it;
 }
 
@@ -135,23 +166,27 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
     __syncthreads();
     tc_fence_after();
     const unsigned tmem = *tmem_slot;
-    const long long lo = ft_bound(p, blockIdx.x), hi = ft_bound(p, blockIdx.x + 1);
+    FtWalk walk = ft_walk(p);
     bool ok = true;
 
     if (warp == 0) {
         if (lane == 0) {
             // the weight boxes of the first stages do not depend on the previous kernel
-            const FtItem first = ft_item(a, p, lo, hi);
+            FtWalk ahead = walk;
+            const FtItem first = ft_next(a, p, ahead);
+            auto load_w = [&](uint8_t* st, const FtItem& it, int b, unsigned long long* bar) {
+                if (p.tiled) tma_load_2d(st, &map_w, 0, (it.wt * p.kb + b) * FT_ROWS, bar);
+                else tma_load_2d(st, &map_w, b * FT_KE, it.pl.n0, bar);
+            };
             const int lead = min(first.nb, STAGES);
             for (int l = 0; l < lead; l++) {
                 mbar_expect_tx(&full[l], Cfg::STAGE_BYTES);
-                tma_load_2d(stages + (size_t)l * Cfg::STAGE_BYTES, &map_w, (first.b0 + l) * FT_KE, first.pl.n0, &full[l]);
+                load_w(stages + (size_t)l * Cfg::STAGE_BYTES, first, first.b0 + l, &full[l]);
             }
             pdl_wait();
             unsigned c = 0;                          // stages issued so far
-            for (long long i = lo; i < hi && ok;) {
-                const FtItem it = ft_item(a, p, i, hi);
-                i += it.nb;
+            while (ft_more(walk) && ok) {
+                const FtItem it = ft_next(a, p, walk);
                 const int row = a.seg_in[it.pl.seg] * p.m_rows + it.tt * TOK;
                 for (int l = 0; l < it.nb; l++, c++) {
                     const int s = c % STAGES;
@@ -160,7 +195,7 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                         ok = mbar_wait(&empty[s], ((c / STAGES) & 1u) ^ 1u, wl);
                         if (!ok) break;
                         mbar_expect_tx(&full[s], Cfg::STAGE_BYTES);
-                        tma_load_2d(st, &map_w, (it.b0 + l) * FT_KE, it.pl.n0, &full[s]);
+                        load_w(st, it, it.b0 + l, &full[s]);
                     }
                     tma_load_2d(st + FT_A_BYTES, &map_x, (it.b0 + l) * FT_KE, row, &full[s]);
                 }
@@ -174,9 +209,8 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
     } else if (warp == 1) {
         if (lane == 0) {
             unsigned c = 0, t = 0;
-            for (long long i = lo; i < hi && ok; t++) {
-                const FtItem it = ft_item(a, p, i, hi);
-                i += it.nb;
+            for (; ft_more(walk) && ok; t++) {
+                const FtItem it = ft_next(a, p, walk);
                 const unsigned b = t & 1u;
                 ok = mbar_wait(&tempty[b], ((t >> 1) & 1u) ^ 1u, wl);
                 if (!ok) break;
@@ -201,9 +235,8 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
         pdl_wait();
         unsigned t = 0;
         constexpr size_t PIECE = (size_t)TOK * FT_ROWS;
-        for (long long i = lo; i < hi && ok; t++) {
-            const FtItem it = ft_item(a, p, i, hi);
-            i += it.nb;
+        for (; ft_more(walk) && ok; t++) {
+            const FtItem it = ft_next(a, p, walk);
             const unsigned b = t & 1u;
             ok = mbar_wait(&tfull[b], (t >> 1) & 1u, wl);
             if (!ok) break;
@@ -234,22 +267,23 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
             if (whole) continue;
             // a piece: the tile's CTAs meet at a counter; the last one adds the pieces
             __shared__ unsigned last_cta;
-            const long long u0 = (long long)it.tile * p.kb;
-            const int first_cta = ft_owner(p, u0), end_cta = ft_owner(p, u0 + p.kb - 1);
+            const long long u0 = (long long)it.wt * p.kb;
+            const int first = ft_owner(p, walk, u0), end = ft_owner(p, walk, u0 + p.kb - 1);   // ranks; CTA = rank * tok_tiles + tt
+            unsigned* counter = p.counters + first * p.tok_tiles + it.tt;
             __threadfence();
             asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
-            if (et == 0) last_cta = atomicAdd(p.counters + first_cta, 1u) == (unsigned)(end_cta - first_cta);
+            if (et == 0) last_cta = atomicAdd(counter, 1u) == (unsigned)(end - first);
             asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");
             if (last_cta) {
                 __threadfence();
-                if (et == 0) p.counters[first_cta] = 0;
+                if (et == 0) *counter = 0;
                 const float* all = p.part + (size_t)col0 * FT_ROWS + q * 32 + lane;
                 for (int c = 0; c < Cfg::EC && m0 + c < a.M; c += 32) {
                     float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; j++) v[j] = 0.0f;
-                    for (int s = first_cta; s <= end_cta; s++) {
-                        const float* piece = all + ((size_t)s * 2 + (s == first_cta ? 1 : 0)) * PIECE + (size_t)c * FT_ROWS;
+                    for (int s = first; s <= end; s++) {
+                        const float* piece = all + ((size_t)(s * p.tok_tiles + it.tt) * 2 + (s == first ? 1 : 0)) * PIECE + (size_t)c * FT_ROWS;
 #pragma unroll
                         for (int j = 0; j < 32; j++) v[j] += __ldcg(piece + (size_t)j * FT_ROWS);
                     }
@@ -289,19 +323,19 @@ static void launch_tok(FgemmArgs a, cudaStream_t q) {
     FtPlan p{};
     p.tok_tiles = (a.M + TOK - 1) / TOK;
     p.kb = (a.K + FT_KE - 1) / FT_KE;
-    p.tiles = a.tile0[a.nseg] * p.tok_tiles;
-    const int sms = sm_count();
-    int grid = std::min(p.tiles, sms);
+    p.wtiles = a.tile0[a.nseg];
+    const int sms = sm_count(), tiles = p.wtiles * p.tok_tiles;
+    int grid = std::min(tiles, sms);
     if (!(float_flags() & 4)) {
-        // deal out stages when whole tiles keep less than 92 % of the SM-rounds busy, and a share is worth the hand-over
-        const long long units = (long long)p.tiles * p.kb;
-        const int rounds = (p.tiles + sms - 1) / sms, share = TOK == 32 ? 6 : 16;
+        // deal out stages when whole tiles keep less than 80 % of the SM-rounds busy, and a share is worth the hand-over
+        const long long units = (long long)tiles * p.kb;
+        const int rounds = (tiles + sms - 1) / sms, share = TOK == 32 ? 6 : 16;
         const int want = (int)std::min<long long>(sms, units / share);
         size_t bytes = 0;
         int ncnt = 0;
         p.part = fsplit_workspace(&bytes);
         p.counters = fsplit_counters(&ncnt);
-        if (p.tiles < 0.92 * rounds * sms && want >= grid && want <= ncnt &&
+        if (tiles < 0.8 * rounds * sms && want >= grid && want >= 2 * p.tok_tiles && want <= ncnt &&
             (size_t)want * 2 * TOK * FT_ROWS * sizeof(float) <= bytes) {
             p.dealt = 1;
             grid = want;
@@ -312,7 +346,8 @@ static void launch_tok(FgemmArgs a, cudaStream_t q) {
     p.m_rows = groups == 1 ? 0 : (int)(a.gstride / a.ldx);
     const size_t x_rows = (size_t)(groups - 1) * p.m_rows + a.M;
     DETB_REQUIRE(a.ldw == round8(a.K), "linear: weight rows must be padded to 8 elements");
-    const CUtensorMap map_w = bf16_map(a.w, a.N, a.ldw, FT_ROWS);
+    p.tiled = a.wt != nullptr;
+    const CUtensorMap map_w = p.tiled ? bf16_map(a.wt, (size_t)p.wtiles * p.kb * FT_ROWS, FT_KE, FT_ROWS) : bf16_map(a.w, a.N, a.ldw, FT_ROWS);
     const CUtensorMap map_x = bf16_map(a.x, x_rows, a.ldx, TOK);
     static bool configured = false;
     if (!configured) {
@@ -322,6 +357,19 @@ static void launch_tok(FgemmArgs a, cudaStream_t q) {
     launch_pdl(k_fgemm_tc<TOK>, dim3(grid), dim3(Cfg::THREADS), Cfg::SMEM, q, 1, map_w, map_x, a, p);
 }
 
+// One 16-byte piece (8 values of a row) per thread.
+__global__ void k_flinear_tile(const FgemmArgs a, int kb, bf16* __restrict__ dst) {
+    const long long id = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    const int per_tile = kb * FT_ROWS * (FT_KE / 8);
+    if (id >= (long long)a.tile0[a.nseg] * per_tile) return;
+    const int t = (int)(id / per_tile), i = (int)(id % per_tile);
+    const int b = i / (FT_ROWS * 8), r = i / 8 % FT_ROWS, k = b * FT_KE + (i & 7) * 8;
+    const TilePlace pl = place_tile<FT_ROWS>(a, t);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (pl.n0 + r < pl.n_end && k < a.ldw) v = *reinterpret_cast<const uint4*>(a.w + (size_t)(pl.n0 + r) * a.ldw + k);
+    reinterpret_cast<uint4*>(dst)[id] = v;
+}
+
 void fgemm_tc_launch(FgemmArgs a, cudaStream_t q) {
     if (a.M <= 32) launch_tok<32>(a, q);
     else if (a.M <= 128) launch_tok<128>(a, q);
@@ -329,3 +377,34 @@ void fgemm_tc_launch(FgemmArgs a, cudaStream_t q) {
 }
 
 }  // namespace detb
+
+using namespace detb;
+
+static FgemmArgs tile_args(int K, int nseg, const int* seg_end) {
+    DETB_REQUIRE(K > 0 && nseg >= 1 && nseg <= 8, "linear: bad segments");
+    FgemmArgs a{};
+    a.K = K;
+    a.nseg = nseg;
+    for (int i = 0; i < nseg; i++) a.seg_end[i] = seg_end[i];
+    plan_tiles(a, FT_ROWS);
+    return a;
+}
+
+extern "C" {
+
+size_t det_f_linear_tile_bytes(int K, int nseg, const int* seg_end) {
+    return (size_t)tile_args(K, nseg, seg_end).tile0[nseg] * ((K + FT_KE - 1) / FT_KE) * FT_A_BYTES;
+}
+void det_f_linear_tile(const det_flinear* src, int nseg, const int* seg_end, void* dst, cudaStream_t st) {
+    FgemmArgs a = tile_args(src->K, nseg, seg_end);
+    DETB_REQUIRE(seg_end[nseg - 1] == src->N && src->ld % 8 == 0, "linear: bad segments");
+    a.w = static_cast<const bf16*>(src->w);
+    a.N = src->N;
+    a.ldw = src->ld;
+    const int kb = (src->K + FT_KE - 1) / FT_KE;
+    const long long n = (long long)a.tile0[nseg] * kb * FT_ROWS * (FT_KE / 8);
+    k_flinear_tile<<<(unsigned)((n + 255) / 256), 256, 0, queue_of(st)>>>(a, kb, static_cast<bf16*>(dst));
+    DETB_CUDA_OK(cudaGetLastError());
+}
+
+}  // extern "C"

@@ -53,6 +53,7 @@ __device__ __forceinline__ int position_of(const det_seq_ref& r, int row) {
 // ---- entries between the translation units
 struct FgemmArgs {
     const bf16* w;
+    const bf16* wt;          // tile-major copy, or NULL
     int N, K, ldw;
     const void* x;
     int ldx;

@@ -134,7 +134,9 @@ inline size_t dtype_bytes(Dtype d) { return d == Dtype::BF16 ? 2 : 4; }
 struct FLinear {
     Buf<uint16_t> w;
     size_t n = 0, k = 0, ld = 0;
-    det_flinear view() const { return det_flinear{w.ptr(), (int)n, (int)k, (int)ld}; }
+    std::vector<int> seg_end;   // rows in segments of their own inputs (det_fgemm_op)
+    Buf<uint16_t> tiles;        // backend's second copy for batches, may be empty (Backend::f_linear_ready)
+    det_flinear view() const { return det_flinear{w.ptr(), (int)n, (int)k, (int)ld, tiles.ptr()}; }
 };
 // What one sequence keeps in one layer; a layer uses the members it needs.
 struct FloatState {
@@ -245,6 +247,7 @@ class Backend {
     virtual std::unique_ptr<RowSet> make_slots(std::vector<const FloatState*>) { no_float_ops(); return nullptr; }
     // The sequence reference of a step: `t` tokens of `st` from pos0 on, or one row per sequence of `rows`.
     virtual det_seq_ref seq_ref(const FloatState&, size_t, const RowSet*, const Buf<int32_t>*) { no_float_ops(); return {}; }
+    virtual void f_linear_ready(FLinear&) {}   // the rows are in place: a backend may add a layout of its own
     virtual void f_norm(const det_fnorm_op&) { no_float_ops(); }
     virtual void f_gemm(const det_fgemm_op&) { no_float_ops(); }
     virtual void f_recur(const det_frecur_op&) { no_float_ops(); }             // the backend supplies `scratch`

@@ -575,6 +575,14 @@ det_seq_ref CudaBackend::seq_ref(const FloatState& st, size_t pos0, const RowSet
     r.pos0 = (int)pos0;
     return r;
 }
+// The tile-major copy that the tensor-core GEMM's loads read (int8_layout: the same switch as for quantized linears).
+void CudaBackend::f_linear_ready(FLinear& l) {
+    if (!int8_layout) return;
+    const int nseg = (int)l.seg_end.size();
+    const det_flinear src = l.view();
+    l.tiles = alloc<uint16_t>(det_f_linear_tile_bytes((int)l.k, nseg, l.seg_end.data()) / 2);
+    det_f_linear_tile(&src, nseg, l.seg_end.data(), l.tiles.ptr(), ST);
+}
 void CudaBackend::f_norm(const det_fnorm_op& op) {
     flush_pending();
     det_f_norm(&op, ST);

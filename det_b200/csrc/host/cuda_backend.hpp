@@ -60,6 +60,7 @@ class CudaBackend : public Backend {
     void embed(const void* table, int type, const Buf<int32_t>& ids, size_t t, size_t h, const Buf<float>& x) override;
     std::unique_ptr<RowSet> make_slots(std::vector<const FloatState*> fs) override;
     det_seq_ref seq_ref(const FloatState& st, size_t pos0, const RowSet* rows, const Buf<int32_t>* pos) override;
+    void f_linear_ready(FLinear& l) override;
     void f_norm(const det_fnorm_op& op) override;
     void f_gemm(const det_fgemm_op& op) override;
     void f_recur(const det_frecur_op& op) override;

@@ -171,7 +171,7 @@ class Packer {
             std::memcpy(&host_[(row0 + r * step) * lin_.ld + col0], &tmp_[r * cols], cols * 2);
         filled_.push_back({row0, step, rows});
     }
-    FLinear finish() {
+    FLinear finish(std::vector<int> seg_end = {}) {
         if (!host_.empty()) {
             size_t lo = lin_.n, hi = 0;   // rows written on the host form one span (device-filled parts lie outside it)
             for (const auto& f : filled_) {
@@ -181,6 +181,9 @@ class Packer {
             bk_->write(lin_.w, lo * lin_.ld, host_.data() + lo * lin_.ld, (hi - lo) * lin_.ld);
             bk_->sync();   // the staging buffer dies here
         }
+        lin_.seg_end = std::move(seg_end);
+        if (lin_.seg_end.empty()) lin_.seg_end = {(int)lin_.n};
+        bk_->f_linear_ready(lin_);
         return std::move(lin_);
     }
 
@@ -236,7 +239,12 @@ static std::shared_ptr<HybridWeights> load_layer(const HybridConfig& c, size_t i
             in.part(mlp + "up", l.ff, W, w.plain + 1, 2);
         }
     }
-    w.in = in.finish();
+    std::vector<int> ends;      // wkv: every part reads an input of its own
+    if (m.kind == MixerKind::Wkv)
+        for (size_t q = 1; q < parts.size(); q++) ends.push_back((int)w.off[q]);
+    ends.push_back((int)w.plain);
+    if (l.ff) ends.push_back((int)(w.plain + 2 * l.ff));
+    w.in = in.finish(ends);
 
     w.out_ff = round8(vo);
     Packer out(bk, src, W, l.ff ? w.out_ff + l.ff : vo);
@@ -454,10 +462,11 @@ void HybridModel::run_in(const LayerSpec& l, const HybridWeights& w, size_t t, c
     g.group_stride = (long long)(max_batch * ld_in_);
     g.M = (int)t;
     g.glu_from = (int)w.plain;
-    auto segment = [&](size_t end, int in) {
-        g.seg_end[g.nseg] = (int)end;
-        g.seg_in[g.nseg++] = in;
-    };
+    g.nseg = (int)w.in.seg_end.size();
+    for (int i = 0; i < g.nseg; i++) {
+        g.seg_end[i] = w.in.seg_end[i];
+        g.seg_in[i] = l.mixer.kind == MixerKind::Wkv ? i : 0;     // r, k, v, g, w1, then the feed-forward on h itself
+    }
     if (l.mixer.kind == MixerKind::Wkv) {
         det_fnorm_op n{};
         n.x = x.ptr();
@@ -473,14 +482,10 @@ void HybridModel::run_in(const LayerSpec& l, const HybridWeights& w, size_t t, c
         n.mu = w.mu.ptr();
         n.seq = seq;
         backend->f_norm(n);
-        for (int p = 0; p < 5; p++) segment(p < 4 ? w.off[p + 1] : w.plain, p);
-        if (l.ff) segment(w.in.n, 5);
     } else {
         g.norm_x = x.ptr();
         g.norm_w = w.norm1.ptr();
         g.eps = cfg.eps;
-        segment(w.plain, 0);
-        if (l.ff) segment(w.in.n, 0);
     }
     g.y = y_.ptr();
     g.ldy = (int)round8(w.plain);

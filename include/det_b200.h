@@ -386,11 +386,17 @@ void det_debug_xchg_drop(void* h, int rank);
 #define DET_F32 0
 #define DET_BF16 1
 
-/* W[N][ld] bfloat16, ld a multiple of 8, columns K..ld zero. */
+/* W[N][ld] bfloat16, ld a multiple of 8, columns K..ld zero.  wt (NULL: none) is a second copy for the tensor-core GEMM whose
+ * TMA boxes are 16 KB of consecutive memory: [row tile][K / 64 rounded up][128 rows][64 values], the row tiles of every
+ * segment starting at its first row and padded with zeros.  det_f_linear_tile builds it for the segments that the calls
+ * will name (seg_end as in det_fgemm_op); det_f_linear_tile_bytes is its size.                                         */
 typedef struct {
     const void* w;
     int N, K, ld;
+    const void* wt;
 } det_flinear;
+size_t det_f_linear_tile_bytes(int K, int nseg, const int* seg_end);
+void det_f_linear_tile(const det_flinear* src, int nseg, const int* seg_end, void* dst, cudaStream_t st);
 
 /* What one sequence keeps in one layer: recurrent state s[heads][dk][dv], the previous token's normalised row prev[n], and
  * a cache of `cap` rows used as a ring (the row of position p is row p % cap).  A layer uses the members it needs.     */

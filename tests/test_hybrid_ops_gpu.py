@@ -142,6 +142,10 @@ def test_products(dtype, flags, m, gpu, libs):
         op = libs.FGemmOp(lin=C.pointer(lin), dtype=code(libs, dtype), x=px, ldx=ld, group_stride=(m + 2) * ld, nseg=len(ends),
                           seg_end=(C.c_int * 8)(*ends), seg_in=(C.c_int * 8)(*ins), glu_from=sum(n_plain), M=m, y=gpu.f32(y0),
                           ldy=sum(n_plain), accumulate=1, h=gpu.space(4 * m * round8(max(ff, 1))), ldh=round8(max(ff, 1)))
+        if m % 2:                                        # with and without the tile-major copy of the weights
+            ends_c = (C.c_int * 8)(*ends)
+            lin.wt = gpu.space(gpu.d.det_f_linear_tile_bytes(k, len(ends), ends_c))
+            gpu.d.det_f_linear_tile(C.byref(lin), len(ends), ends_c, lin.wt, None)
         gpu.d.det_debug_set_float(flags)
         try:
             gpu.d.det_f_gemm(C.byref(op), None)
