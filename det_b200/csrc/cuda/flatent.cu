@@ -338,6 +338,13 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const unsigned (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+// 2^x by the special function unit (relative error about 2^-22; 2^-inf = 0).
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // One head x 64 query rows; DV = value dimensions rounded up to a multiple of 64.
 template <int DV>
 __global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentArgs a) {
@@ -368,45 +375,43 @@ __global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentA
     }
     const bf16* cache = static_cast<const bf16*>(a.seq.one.cache);
     const int kvec = a.dim / 8, rvec = a.rot_dim / 8, vvec = a.vdim / 8, tvec = kvec + rvec + vvec;
-    // a warp copies whole key rows; which pieces of a row a lane takes does not depend on the row
+    // a warp copies whole key rows; which 16-byte pieces of a row a lane takes does not depend on the row
     constexpr int PIECES = 3;
     const bf16* piece[PIECES];
-    size_t step[PIECES];
-    bf16* to[PIECES];
-    int ldt[PIECES];
+    int step[PIECES];
+    unsigned to[PIECES], ldt[PIECES];
 #pragma unroll
     for (int j = 0; j < PIECES; j++) {
         const int v = lane + j * 32;
         piece[j] = nullptr;
-        step[j] = 0;
-        to[j] = Kt;
-        ldt[j] = ldk;
+        step[j] = a.ldkv;
+        to[j] = 0;
+        ldt[j] = ldk * 2;
         if (v < kvec) {
             piece[j] = a.kv + h * a.dim + v * 8;
-            step[j] = a.ldkv;
-            to[j] = Kt + v * 8;
+            to[j] = smem_addr(Kt + v * 8);
         } else if (v < kvec + rvec) {
             piece[j] = cache + a.rp + (v - kvec) * 8;
             step[j] = a.ld;
-            to[j] = Kt + v * 8;
+            to[j] = smem_addr(Kt + v * 8);
         } else if (v < tvec) {
             piece[j] = a.kv + a.heads * a.dim + h * a.vdim + (v - kvec - rvec) * 8;
-            step[j] = a.ldkv;
-            to[j] = Vt + (v - kvec - rvec) * 8;
-            ldt[j] = LDV;
+            to[j] = smem_addr(Vt + (v - kvec - rvec) * 8);
+            ldt[j] = LDV * 2;
         }
     }
     auto fetch = [&](int k0, int buf) {
-        const int slot0 = k0 % a.cap;
-        for (int k = warp; k < FL_KEYS; k += FL_WARPS) {
-            int slot = slot0 + min(k, p_last - k0);               // past the last key: a copy of it, masked below
-            while (slot >= a.cap) slot -= a.cap;
+        const int slot0 = k0 % a.cap, last = p_last - k0;         // past the last key: a copy of it, masked below
 #pragma unroll
-            for (int j = 0; j < PIECES; j++)
-                if (piece[j])
-                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(to[j] + (buf * FL_KEYS + k) * ldt[j])),
-                                 "l"(piece[j] + (size_t)slot * step[j])
-                                 : "memory");
+        for (int j = 0; j < PIECES; j++) {
+            if (!piece[j]) continue;
+            unsigned dst = to[j] + (unsigned)(buf * FL_KEYS + warp) * ldt[j];
+#pragma unroll 4
+            for (int k = warp; k < FL_KEYS; k += FL_WARPS, dst += FL_WARPS * ldt[j]) {
+                int slot = slot0 + min(k, last);
+                if (slot >= a.cap) slot = a.cap >= FL_KEYS ? slot - a.cap : slot % a.cap;
+                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(piece[j] + (long long)slot * step[j]) : "memory");
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -437,6 +442,7 @@ __global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentA
             for (int i = 0; i < 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
             const bf16* K = Kt + (size_t)buf * FL_KEYS * ldk;
             const unsigned kaddr = smem_addr(K + ((lane & 7) + ((lane >> 4) << 3)) * ldk + ((lane >> 3) & 1) * 8);
+#pragma unroll 2
             for (int kk = 0; kk < dqp; kk += 16) {
                 unsigned qa[4];
                 ldsm4(qaddr + kk * 2, qa);
@@ -473,22 +479,24 @@ __global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentA
 #pragma unroll
             for (int i = 0; i < 2; i++) {
                 base[i] = mx[i] == -INFINITY ? 0.0f : mx[i];       // no key seen yet: every weight below is exp2(-inf) = 0
-                f[i] = exp2f(m[i] - base[i]);
+                f[i] = exp2_fast(m[i] - base[i]);
                 m[i] = mx[i];
                 l[i] *= f[i];
             }
+            if (__any_sync(FULL, f[0] != 1.0f || f[1] != 1.0f)) {
 #pragma unroll
-            for (int i = 0; i < DV / 8; i++) {
-                o[i][0] *= f[0];
-                o[i][1] *= f[0];
-                o[i][2] *= f[1];
-                o[i][3] *= f[1];
+                for (int i = 0; i < DV / 8; i++) {
+                    o[i][0] *= f[0];
+                    o[i][1] *= f[0];
+                    o[i][2] *= f[1];
+                    o[i][3] *= f[1];
+                }
             }
             unsigned pf[4][4];
 #pragma unroll
             for (int n = 0; n < 8; n++) {
-                const float e0 = exp2f(s[n][0] - base[0]), e1 = exp2f(s[n][1] - base[0]);
-                const float e2 = exp2f(s[n][2] - base[1]), e3 = exp2f(s[n][3] - base[1]);
+                const float e0 = exp2_fast(s[n][0] - base[0]), e1 = exp2_fast(s[n][1] - base[0]);
+                const float e2 = exp2_fast(s[n][2] - base[1]), e3 = exp2_fast(s[n][3] - base[1]);
                 l[0] += e0 + e1;
                 l[1] += e2 + e3;
                 pf[n >> 1][(n & 1) * 2] = pack_bf(e0, e1);

@@ -5,7 +5,7 @@
 //                   with a slab of the head's columns, computes the decays from their low-rank projection, streams the state
 //                   once, exchanges the sums of squares over distributed shared memory and finishes with the head's RMS norm
 //                   and gate, so a layer step is one launch.  Bound by the bytes of the states.
-//   k_frecur_scan   a run of tokens of one sequence: a lane keeps RPL rows of four columns of S in registers, PARTS lanes share
+//   k_frecur_scan   a run of tokens of one sequence: a lane keeps RPL rows of two columns of S in registers, PARTS lanes share
 //                   the columns; per-token operands arrive in shared memory by asynchronous copies, a block of tokens ahead.
 //                   Bound by the issue of its multiply-adds, three per state element and token.  The decays come from
 //                   k_fdecay, the norm and the gate from k_frecur_out.
@@ -138,7 +138,7 @@ __global__ void __launch_bounds__(RS_THREADS) k_frecur_step(const RecurArgs a, i
 }
 
 // ------------------------------------------------------------------------------------------------------ a run of tokens
-constexpr int SC_WARPS = 2, SC_THREADS = SC_WARPS * 32, SC_TB = 16, SC_CPL = 4;   // tokens per staged block, columns per lane
+constexpr int SC_WARPS = 4, SC_THREADS = SC_WARPS * 32, SC_TB = 16, SC_CPL = 2;   // tokens per staged block, columns per lane
 
 // Asynchronous copy of V floats to shared memory; zeros when `in` is false.
 template <int V>
@@ -161,25 +161,38 @@ __global__ void __launch_bounds__(SC_THREADS) k_frecur_scan(const RecurArgs a) {
     const int col = (warp * LC + lane / PARTS) * SC_CPL;     // first column of this lane inside the CTA
     pdl_trigger();
     pdl_wait();
+    // a thread copies the same one or two elements of every token: pointers advance by a token
+    constexpr int SLOTS = (TOK / V + SC_THREADS - 1) / SC_THREADS;
+    const float* src0[SLOTS];
+    int step[SLOTS];
+    bool in[SLOTS];
+#pragma unroll
+    for (int i = 0; i < SLOTS; i++) {
+        const int e = (threadIdx.x + i * SC_THREADS) * V;
+        src0[i] = nullptr;
+        step[i] = a.ldy;
+        in[i] = false;
+        if (e < 3 * ROWS) {
+            const int which = e / ROWS, r = e % ROWS;
+            in[i] = r < dk;
+            src0[i] = which == 2 ? a.z + (size_t)h * dk : a.y + (which ? a.k_off : a.q_off) + h * dk;
+            if (which == 2) step[i] = a.heads * dk;
+            src0[i] += in[i] ? r : 0;
+        } else if (e < TOK) {
+            const int c = c0 + e - 3 * ROWS;
+            in[i] = c < dv;
+            src0[i] = a.y + a.v_off + h * dv + (in[i] ? c : 0);
+        }
+    }
     auto stage = [&](int t0, int buf) {
-        float* base = scm + buf * (SC_TB * TOK);
         const int nt = min(SC_TB, a.M - t0);
-        for (int i = threadIdx.x; i < nt * (TOK / V); i += SC_THREADS) {
-            const int t = i / (TOK / V), e = (i % (TOK / V)) * V;
-            const float* y = a.y + (size_t)(t0 + t) * a.ldy;
-            const float* src;
-            bool in;
-            if (e < 3 * ROWS) {
-                const int which = e / ROWS, r = e % ROWS;
-                in = r < dk;
-                src = which == 2 ? a.z + ((size_t)(t0 + t) * a.heads + h) * dk : y + (which ? a.k_off : a.q_off) + h * dk;
-                src += in ? r : 0;
-            } else {
-                const int c = c0 + e - 3 * ROWS;
-                in = c < dv;
-                src = y + a.v_off + h * dv + (in ? c : 0);
-            }
-            copy_async<V>(base + t * TOK + e, src, in);
+#pragma unroll
+        for (int i = 0; i < SLOTS; i++) {
+            if (!src0[i]) continue;
+            const float* src = src0[i] + (size_t)t0 * step[i];
+            float* dst = scm + buf * (SC_TB * TOK) + (threadIdx.x + i * SC_THREADS) * V;
+#pragma unroll 4
+            for (int t = 0; t < nt; t++, src += step[i], dst += TOK) copy_async<V>(dst, src, in[i]);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -193,11 +206,11 @@ __global__ void __launch_bounds__(SC_THREADS) k_frecur_scan(const RecurArgs a) {
 #pragma unroll
         for (int c = 0; c < SC_CPL; c++) s[i][c] = (r < dk && c0 + col + c < dv) ? S[(size_t)r * dv + c0 + col + c] : 0.0f;
     }
-    // which of its four columns a lane ends up with after the reduction below, and whether it stores it
-    constexpr int HI = PARTS / 2, LO = PARTS / 4;
-    const bool up = part & HI, up2 = part & LO;
-    const int mine = c0 + col + (up ? 2 : 0) + (up2 ? 1 : 0);
-    const bool stores = (part & (LO - 1)) == 0 && mine < dv;
+    // which of its two columns a lane ends up with after the reduction below, and whether it stores it
+    constexpr int HI = PARTS / 2;
+    const bool up = part & HI;
+    const int mine = c0 + col + (up ? 1 : 0);
+    const bool stores = (part & (HI - 1)) == 0 && mine < dv;
     float* out = a.o + (size_t)h * dv + mine;
     const size_t ldo = (size_t)a.heads * dv;
     for (int t0 = 0, p = 0; t0 < a.M; t0 += SC_TB, p ^= 1) {
@@ -212,9 +225,9 @@ __global__ void __launch_bounds__(SC_THREADS) k_frecur_scan(const RecurArgs a) {
         const float* d = scm + p * (SC_TB * TOK);
 #pragma unroll 2
         for (int t = 0; t < nt; t++, d += TOK) {
-            const float4 v4 = *reinterpret_cast<const float4*>(d + 3 * ROWS + col);
-            const float v[SC_CPL] = {v4.x, v4.y, v4.z, v4.w};
-            float o[SC_CPL] = {0.0f, 0.0f, 0.0f, 0.0f}, b = 0.0f;
+            const float2 v2 = *reinterpret_cast<const float2*>(d + 3 * ROWS + col);
+            const float v[SC_CPL] = {v2.x, v2.y};
+            float o[SC_CPL] = {0.0f, 0.0f}, b = 0.0f;
 #pragma unroll
             for (int i4 = 0; i4 < RPL / 4; i4++) {
                 const float4 q4 = reinterpret_cast<const float4*>(d)[i4 * PARTS + part];
@@ -237,12 +250,10 @@ __global__ void __launch_bounds__(SC_THREADS) k_frecur_scan(const RecurArgs a) {
 #pragma unroll
                 for (int c = 0; c < SC_CPL; c++) o[c] = fmaf(b, v[c], o[c]);     // the sum over parts completes b as well
             }
-            // four sums over PARTS lanes: halve the columns twice, then fold what is left
-            float x = (up ? o[2] : o[0]) + __shfl_xor_sync(FULL, up ? o[0] : o[2], HI);
-            float z = (up ? o[3] : o[1]) + __shfl_xor_sync(FULL, up ? o[1] : o[3], HI);
-            x = (up2 ? z : x) + __shfl_xor_sync(FULL, up2 ? x : z, LO);
+            // two sums over PARTS lanes: one column per half, then fold
+            float x = (up ? o[1] : o[0]) + __shfl_xor_sync(FULL, up ? o[0] : o[1], HI);
 #pragma unroll
-            for (int off = LO / 2; off > 0; off >>= 1) x += __shfl_xor_sync(FULL, x, off);
+            for (int off = HI / 2; off > 0; off >>= 1) x += __shfl_xor_sync(FULL, x, off);
             if (stores) out[(size_t)(t0 + t) * ldo] = x * a.q_scale;
         }
         __syncthreads();
@@ -287,10 +298,10 @@ static void launch_scan(const RecurArgs& a, cudaStream_t q) {
 }
 template <bool BONUS, int V>
 static void scan(const RecurArgs& a, cudaStream_t q) {
-    if (a.dk <= 32) launch_scan<4, 8, BONUS, V>(a, q);
-    else if (a.dk <= 64) launch_scan<8, 8, BONUS, V>(a, q);
+    if (a.dk <= 32) launch_scan<8, 4, BONUS, V>(a, q);
+    else if (a.dk <= 64) launch_scan<16, 4, BONUS, V>(a, q);
     else if (a.dk <= 128) launch_scan<16, 8, BONUS, V>(a, q);
-    else if (a.dk <= 256) launch_scan<16, 16, BONUS, V>(a, q);
+    else if (a.dk <= 256) launch_scan<32, 8, BONUS, V>(a, q);
     else launch_scan<32, 16, BONUS, V>(a, q);
 }
 template <int V>
