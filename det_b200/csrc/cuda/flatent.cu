@@ -364,14 +364,24 @@ __global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentA
     pdl_wait();
     const int p0 = position_of(a.seq, r0), p_last = p0 + nrows - 1;
     const float qs = a.scale * 1.4426950408889634f;                // scores in units of log 2
-    for (int i = threadIdx.x; i < FL_ROWS * dqp; i += NT) {
-        const int r = i / dqp, e = i % dqp;
-        float v = 0.0f;
-        if (r < nrows && e < hd) {
-            const float* q = a.q + (size_t)(r0 + r) * a.ldq + h * hd;
-            v = (e < a.dim ? q[e] : rotated(q + a.dim, e - a.dim, p0 + r, a)) * qs;
+#pragma unroll 4
+    for (int r = warp; r < FL_ROWS; r += FL_WARPS) {               // a warp per row, two neighbouring elements per lane
+        const float* q = a.q + (size_t)(r0 + min(r, nrows - 1)) * a.ldq + h * hd;
+        for (int e = lane * 2; e < dqp; e += 64) {
+            float u = 0.0f, v = 0.0f;
+            if (r < nrows && e < hd) {                             // dim and rot_dim are multiples of 8: pairs do not straddle
+                u = q[e];
+                v = q[e + 1];
+                const int er = e - a.dim;
+                if (er >= 0 && er < a.rot_dims) {
+                    const size_t at = (size_t)(p0 + r) * (a.rot_dims / 2) + (er >> 1);
+                    const float c = a.rope_cos[at], s = a.rope_sin[at], x = u;
+                    u = fmaf(x, c, -(v * s));
+                    v = fmaf(v, c, x * s);
+                }
+            }
+            *reinterpret_cast<unsigned*>(Q + r * ldk + e) = pack_bf(u * qs, v * qs);
         }
-        put(Q + r * ldk + e, v);
     }
     const bf16* cache = static_cast<const bf16*>(a.seq.one.cache);
     const int kvec = a.dim / 8, rvec = a.rot_dim / 8, vvec = a.vdim / 8, tvec = kvec + rvec + vvec;
@@ -588,7 +598,7 @@ static void launch_flash(const LatentArgs& a, cudaStream_t q) {
         DETB_CUDA_OK(cudaFuncSetAttribute(k_latent_flash<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = smem;
     }
-    launch_pdl(k_latent_flash<DV>, dim3((a.M + FL_ROWS - 1) / FL_ROWS, a.heads), dim3(FL_WARPS * 32), smem, q, 1, a);
+    launch_plain(k_latent_flash<DV>, dim3((a.M + FL_ROWS - 1) / FL_ROWS, a.heads), dim3(FL_WARPS * 32), smem, q, a);
 }
 
 static LatentArgs latent_args(const det_flatent_op* op) {

@@ -294,7 +294,7 @@ static void launch_scan(const RecurArgs& a, cudaStream_t q) {
         DETB_CUDA_OK(cudaFuncSetAttribute(k_frecur_scan<PARTS, RPL, BONUS, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = true;
     }
-    launch_pdl(k_frecur_scan<PARTS, RPL, BONUS, V>, dim3((a.dv + COLS - 1) / COLS, a.heads), dim3(SC_THREADS), smem, q, 1, a);
+    launch_plain(k_frecur_scan<PARTS, RPL, BONUS, V>, dim3((a.dv + COLS - 1) / COLS, a.heads), dim3(SC_THREADS), smem, q, a);
 }
 template <bool BONUS, int V>
 static void scan(const RecurArgs& a, cudaStream_t q) {

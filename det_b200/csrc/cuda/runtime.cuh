@@ -65,6 +65,18 @@ inline void launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t s
     DETB_CUDA_OK(launch_pdl_try(kernel, grid, block, smem, q, cluster_x, static_cast<Args&&>(args)...));
 }
 
+// A launch without that attribute: the kernel comes up on an idle device.  For long kernels whose CTAs must spread evenly over
+// the SMs — under programmatic launch they would pile up where the predecessor's first CTAs have left.
+template <class... KArgs, class... Args>
+inline void launch_plain(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t q, Args&&... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = q;
+    DETB_CUDA_OK(cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...));
+}
+
 // Error codes reported by det_last_error().
 enum : int { DETB_ERR_NONE = 0, DETB_ERR_WAIT_EXPIRED = 1, DETB_ERR_SIZE = 2 };
 }  // namespace detb
