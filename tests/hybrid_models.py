@@ -29,7 +29,7 @@ def again(entry, of):
     return {**entry, "weights_of": of}
 
 
-def config(width, vocab, layers, eps=1e-5, softcap=30.0):
+def config(width, vocab, layers, eps=2e-5, softcap=25.0):
     return {"architecture": "Fazilorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "logit_softcap": softcap, "layers": layers}
 
 
