@@ -80,7 +80,7 @@ class FGemmOp(C.Structure):
                 ("group_stride", C.c_longlong), ("nseg", c_int), ("seg_end", c_int * 8), ("seg_in", c_int * 8),
                 ("glu_from", c_int), ("M", c_int), ("norm_x", c_void_p), ("norm_w", c_void_p), ("eps", c_float),
                 ("y", c_void_p), ("ldy", c_int), ("y_bf16", c_int), ("accumulate", c_int), ("softcap", c_float),
-                ("h", c_void_p), ("ldh", c_int)]
+                ("h", c_void_p), ("ldh", c_int), ("bias", c_void_p), ("act", c_int)]
 
 
 class FRecurOp(C.Structure):
@@ -100,7 +100,35 @@ class FLatentOp(C.Structure):
                 ("seq", SeqRef)]
 
 
+class FSeamOp(C.Structure):
+    _fields_ = [("x", c_void_p), ("M", c_int), ("n", c_int), ("eps", c_float), ("y", c_void_p), ("ldy", c_int),
+                ("y_norm", c_void_p), ("y_scale", c_void_p), ("w", c_void_p), ("conv", c_void_p), ("taps", c_int),
+                ("rstd", c_void_p), ("dtype", c_int), ("out", c_void_p), ("ld", c_int), ("seq", SeqRef)]
+
+
+class FAttnOp(C.Structure):
+    _fields_ = [(n, c_int) for n in ("heads", "kv_heads", "dim", "vdim", "rot_dims")] + [
+                ("scale", c_float), ("cap", c_int), ("M", c_int), ("dtype", c_int), ("y", c_void_p), ("ldy", c_int),
+                ("q_off", c_int), ("k_off", c_int), ("v_off", c_int), ("gate_off", c_int), ("rope_cos", c_void_p),
+                ("rope_sin", c_void_p), ("vrope_cos", c_void_p), ("vrope_sin", c_void_p), ("q", c_void_p),
+                ("out", c_void_p), ("ldo", c_int), ("max_pos", c_int), ("scratch", c_void_p), ("seq", SeqRef)]
+
+
+class FMinGruOp(C.Structure):
+    _fields_ = [("n", c_int), ("M", c_int), ("dtype", c_int), ("y", c_void_p), ("ldy", c_int), ("z_off", c_int),
+                ("x_off", c_int), ("gate_off", c_int), ("out", c_void_p), ("ldo", c_int), ("seq", SeqRef)]
+
+
+class FMoeOp(C.Structure):
+    _fields_ = [(n, c_int) for n in ("experts", "identity", "top", "ff", "n", "M", "dtype")] + [
+                ("z", c_void_p), ("ldz", c_int), ("correction", c_void_p), ("x", c_void_p), ("ldx", c_int),
+                ("up", C.POINTER(FLinear)), ("down", C.POINTER(FLinear)), ("shared", C.POINTER(FLinear)),
+                ("hs", c_void_p), ("ldhs", c_int), ("shared_gate", c_int), ("out", c_void_p), ("ldo", c_int),
+                ("counts", c_void_p), ("scratch", c_void_p)]
+
+
 DET_F32, DET_BF16 = 0, 1
+DET_FF_SWIGLU, DET_FF_REGLU, DET_FF_RELU2 = 0, 1, 2
 DET_DECAY_SIGMOID, DET_DECAY_EXP = 0, 1
 DET_LAYOUT_STREAM = 0x100
 DET_LAYOUT_INT8 = 0x200
@@ -193,6 +221,17 @@ CUDA_ABI = {
     "det_f_latent_scratch_bytes": (c_size_t, [c_int] * 10),
     "det_f_latent_prep": (None, [C.POINTER(FLatentOp), c_void_p]),
     "det_f_latent_attn": (None, [C.POINTER(FLatentOp), c_void_p]),
+    "det_f_linear_tile_groups_bytes": (c_size_t, [c_int, c_int, c_int]),
+    "det_f_linear_tile_groups": (None, [C.POINTER(FLinear), c_int, c_void_p, c_void_p]),
+    "det_f_seam": (None, [C.POINTER(FSeamOp), c_void_p]),
+    "det_f_attn_ld": (c_int, [c_int, c_int, c_int]),
+    "det_f_attn_q_ld": (c_int, [c_int, c_int]),
+    "det_f_attn_scratch_bytes": (c_size_t, [c_int]),
+    "det_f_attn_prep": (None, [C.POINTER(FAttnOp), c_void_p]),
+    "det_f_attn": (None, [C.POINTER(FAttnOp), c_void_p]),
+    "det_f_mingru": (None, [C.POINTER(FMinGruOp), c_void_p]),
+    "det_f_moe_scratch_bytes": (c_size_t, [c_int] * 6),
+    "det_f_moe": (None, [C.POINTER(FMoeOp), c_void_p]),
     "det_debug_set_float": (None, [c_int]),
     "det_attn_set_workspace": (None, [c_void_p, c_size_t]),
     "det_debug_set_attn_tc": (None, [c_int, c_int]),

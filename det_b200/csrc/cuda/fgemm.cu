@@ -55,21 +55,34 @@ __device__ __forceinline__ void simt_tile(const bf16* w, int ldw, int n0, int n_
 __global__ void __launch_bounds__(SG_THREADS) k_fgemm_simt(const FgemmArgs a) {
     pdl_trigger();
     pdl_wait();
-    const TilePlace pl = place_tile<SG_N>(a, blockIdx.x);
-    const int t0 = blockIdx.y * SG_M;
+    TilePlace pl;
+    int t0 = blockIdx.y * SG_M, t_end = a.M, n_base = 0;
+    if (a.group_rows) {
+        if ((int)blockIdx.y >= *a.nwork) return;
+        const int4 w = a.work[blockIdx.y];
+        n_base = w.x * a.group_rows;
+        pl = TilePlace{0, n_base + (int)blockIdx.x * SG_N, n_base + a.group_rows};
+        t0 = w.y;
+        t_end = w.z;
+    } else {
+        pl = place_tile<SG_N>(a, blockIdx.x);
+    }
     const float* x = static_cast<const float*>(a.x) + (size_t)a.seg_in[pl.seg] * a.gstride;
     float acc[4][4];
-    simt_tile(a.w, a.ldw, pl.n0, pl.n_end, a.K, t0, a.M, [&](int t, int k) { return x[(size_t)t * a.ldx + k]; }, acc);
+    simt_tile(a.w, a.ldw, pl.n0, pl.n_end, a.K, t0, t_end, [&](int t, int k) { return x[(size_t)t * a.ldx + k]; }, acc);
     const int tr = threadIdx.x & 15, tc = threadIdx.x >> 4;
 #pragma unroll
     for (int t = 0; t < 4; t++) {
         const int m = t0 + tc * 4 + t;
-        if (m >= a.M) continue;
+        if (m >= t_end) continue;
         if (pl.n0 >= a.glu_from) {
+            float* h = static_cast<float*>(a.h) + (size_t)m * a.ldh;
 #pragma unroll
-            for (int r = 0; r < 4; r += 2) {
+            for (int r = 0; r < 4; r++) {
                 const int n = pl.n0 + tr * 4 + r;
-                if (n < pl.n_end) static_cast<float*>(a.h)[(size_t)m * a.ldh + (n - a.glu_from) / 2] = silu_fast(acc[r][t]) * acc[r + 1][t];
+                if (n >= pl.n_end) continue;
+                if (a.act == DET_FF_RELU2) h[n - n_base - a.glu_from] = relu_squared(acc[r][t]);
+                else if (!(r & 1)) h[(n - a.glu_from) / 2] = gate_pair(a.act, acc[r][t], acc[r | 1][t]);
             }
             continue;
         }
@@ -78,8 +91,9 @@ __global__ void __launch_bounds__(SG_THREADS) k_fgemm_simt(const FgemmArgs a) {
             const int n = pl.n0 + tr * 4 + r;
             if (n >= pl.n_end) continue;
             float v = acc[r][t];
+            if (a.bias) v += a.bias[n];
             if (a.softcap > 0.0f) v = a.softcap * tanhf(v / a.softcap);
-            const size_t at = (size_t)m * a.ldy + n;
+            const size_t at = (size_t)m * a.ldy + n - n_base;
             if (a.yb) put(a.yb + at, v);
             else a.y[at] = a.accumulate ? a.y[at] + v : v;
         }
@@ -110,6 +124,19 @@ __global__ void __launch_bounds__(SG_THREADS) k_fdecay(const DecayArgs a) {
 void fgemm_simt_launch(FgemmArgs a, cudaStream_t q) {
     plan_tiles(a, SG_N);
     launch_pdl(k_fgemm_simt, dim3(a.tile0[a.nseg], (a.M + SG_M - 1) / SG_M), dim3(SG_THREADS), 0, q, 1, a);
+}
+
+// Token tiles of a work list: enough rows for what a linear of the stack gets on average.
+int fgemm_group_tok(int dtype, int rows) {
+    if (dtype != DET_BF16) return SG_M;
+    return rows <= 24 ? 32 : 128;
+}
+void fgemm_group_launch(FgemmArgs a, int dtype, int tok, cudaStream_t q) {
+    if (dtype == DET_BF16) {
+        fgemm_tc_group_launch(a, tok, q);
+        return;
+    }
+    launch_pdl(k_fgemm_simt, dim3((a.group_rows + SG_N - 1) / SG_N, a.max_work), dim3(SG_THREADS), 0, q, 1, a);
 }
 
 void fdecay_launch(const det_flinear* w2, const float* low, int ldlow, const float* bias, int kind, float tau, int M, float* z,
@@ -148,7 +175,7 @@ extern "C" void det_f_gemm(const det_fgemm_op* op, cudaStream_t st) {
         DETB_REQUIRE(op->seg_end[i] > start && op->seg_in[i] >= 0, "linear: bad segments");
         DETB_REQUIRE(!op->norm_x || op->seg_in[i] == 0, "linear: a normalised input has one group");
         glu_ok = glu_ok || start == op->glu_from;
-        DETB_REQUIRE(start < op->glu_from || (op->seg_end[i] - start) % 2 == 0, "linear: an odd number of pair rows");
+        DETB_REQUIRE(start < op->glu_from || op->act == DET_FF_RELU2 || (op->seg_end[i] - start) % 2 == 0, "linear: an odd number of pair rows");
         start = op->seg_end[i];
     }
     DETB_REQUIRE(glu_ok, "linear: the pair rows must start a segment");
@@ -163,6 +190,9 @@ extern "C" void det_f_gemm(const det_fgemm_op* op, cudaStream_t st) {
     a.accumulate = op->accumulate;
     a.softcap = op->softcap;
     a.h = op->h; a.ldh = op->ldh;
+    a.bias = op->bias;
+    a.act = op->act;
+    DETB_REQUIRE(op->act >= DET_FF_SWIGLU && op->act <= DET_FF_RELU2, "linear: unknown activation");
     a.error_flag = error_word();
     cudaStream_t q = queue_of(st);
     if (op->norm_x) {

@@ -8,6 +8,9 @@
 // When whole tiles would leave SMs idle in the last round, the stages of all tiles are dealt out evenly instead: a CTA may then
 // begin or end inside a tile.  Such a piece goes to the library's workspace, and the CTA that arrives last at the tile adds
 // its pieces in order of K, so the result does not depend on the order of arrival.
+//
+// Over a stack of linears (a mixture's experts) the token tiles come from a work list in device memory: a tile then is
+// (entry, weight tile of the entry's linear), whole tiles are dealt round robin, and input rows are already sorted by linear.
 #include "umma.cuh"
 #include "fops.cuh"
 #include <algorithm>
@@ -34,6 +37,7 @@ struct FtPlan {
     int tok_tiles, wtiles, kb;            // token tiles, weight tiles, stages over the whole of K
     int tiled;                            // weights come from the tile-major copy
     int dealt;                            // stages are dealt out evenly (else whole tiles)
+    int grouped;                          // tiles come from FgemmArgs.work; wtiles is per linear
     int m_rows;                           // rows of one input group in the tensor map
     float* part;                          // [CTA][2][TOK][FT_ROWS]: the piece that continues a tile, the piece that begins one
     unsigned* counters;                   // one per CTA that begins a shared tile
@@ -55,6 +59,8 @@ __device__ __forceinline__ void umma_bf16(unsigned tmem_d, unsigned long long da
 struct FtItem {
     TilePlace pl;
     int wt, tt, b0, nb;                   // weight tile, token tile, first stage and number of stages
+    int x_row, m0, m_end;                 // first row in the tensor map; output rows of the tile
+    int n_base;                           // row of W whose output is column 0
 };
 struct FtWalk {
     long long u, hi;                      // dealt: stage positions; else tile numbers
@@ -63,12 +69,12 @@ struct FtWalk {
 __device__ __forceinline__ long long ft_bound(const FtPlan& p, const FtWalk& w, int rank) {
     return (long long)rank * p.wtiles * p.kb / w.ctas;
 }
-__device__ __forceinline__ FtWalk ft_walk(const FtPlan& p) {
+__device__ __forceinline__ FtWalk ft_walk(const FgemmArgs& a, const FtPlan& p) {
     FtWalk w;
     w.ctas = w.rank = 0;
     if (!p.dealt) {
         w.u = blockIdx.x;
-        w.hi = (long long)p.wtiles * p.tok_tiles;
+        w.hi = (long long)p.wtiles * (p.grouped ? *a.nwork : p.tok_tiles);
         return w;
     }
     const int tt = blockIdx.x % p.tok_tiles;
@@ -86,8 +92,24 @@ __device__ __forceinline__ int ft_owner(const FtPlan& p, const FtWalk& w, long l
     return c;
 }
 __device__ __forceinline__ bool ft_more(const FtWalk& w) { return w.u < w.hi; }
+template <int TOK>
 __device__ __forceinline__ FtItem ft_next(const FgemmArgs& a, const FtPlan& p, FtWalk& w) {
     FtItem it;
+    it.n_base = 0;
+    if (p.grouped) {
+        it.tt = (int)(w.u / p.wtiles);
+        const int wt = (int)(w.u - (long long)it.tt * p.wtiles);
+        const int4 e = a.work[it.tt];
+        it.n_base = e.x * a.group_rows;
+        it.wt = e.x * p.wtiles + wt;
+        it.b0 = 0;
+        it.nb = p.kb;
+        it.pl = TilePlace{0, it.n_base + wt * FT_ROWS, it.n_base + a.group_rows};
+        it.x_row = it.m0 = e.y;
+        it.m_end = e.z;
+        w.u += gridDim.x;
+        return it;
+    }
     if (p.dealt) {
         it.wt = (int)(w.u / p.kb);
         it.tt = blockIdx.x % p.tok_tiles;
@@ -102,36 +124,52 @@ __device__ __forceinline__ FtItem ft_next(const FgemmArgs& a, const FtPlan& p, F
         w.u += gridDim.x;
     }
     it.pl = place_tile<FT_ROWS>(a, it.wt);
+    it.m0 = it.tt * TOK;
+    it.m_end = a.M;
+    it.x_row = a.seg_in[it.pl.seg] * p.m_rows + it.m0;
     return it;
 }
 
 // Two neighbouring tokens (columns) of one weight row: v0 at token m, v1 at token m + 1.
-__device__ __forceinline__ void ft_emit2(const FgemmArgs& a, const TilePlace& pl, int n, int m, float v0, float v1) {
+__device__ __forceinline__ void ft_emit2(const FgemmArgs& a, const FtItem& it, int n, int m, float v0, float v1) {
+    const TilePlace& pl = it.pl;
     if (pl.n0 >= a.glu_from) {
+        if (a.act == DET_FF_RELU2) {
+            if (n >= pl.n_end) return;
+            bf16* h = static_cast<bf16*>(a.h) + (size_t)m * a.ldh + (n - it.n_base - a.glu_from);
+            if (m < it.m_end) put(h, relu_squared(v0));
+            if (m + 1 < it.m_end) put(h + a.ldh, relu_squared(v1));
+            return;
+        }
         // lanes 2i / 2i + 1 hold gate / up: the even lane takes token m, the odd one token m + 1
         const bool odd = threadIdx.x & 1;
         const float got = __shfl_xor_sync(FULL, odd ? v0 : v1, 1);
         const float g = odd ? got : v0, u = odd ? v1 : got;
         const int mm = m + (odd ? 1 : 0);
-        if (n < pl.n_end && mm < a.M)
-            put(static_cast<bf16*>(a.h) + (size_t)mm * a.ldh + (n - a.glu_from) / 2, silu_fast(g) * u);
+        if (n < pl.n_end && mm < it.m_end)
+            put(static_cast<bf16*>(a.h) + (size_t)mm * a.ldh + (n - a.glu_from) / 2, gate_pair(a.act, g, u));
         return;
     }
     if (n >= pl.n_end) return;
+    if (a.bias) {
+        const float b = a.bias[n];
+        v0 += b;
+        v1 += b;
+    }
     if (a.softcap > 0.0f) {
         v0 = a.softcap * tanhf(v0 / a.softcap);
         v1 = a.softcap * tanhf(v1 / a.softcap);
     }
-    const size_t at = (size_t)m * a.ldy + n;
+    const size_t at = (size_t)m * a.ldy + n - it.n_base;
     if (a.yb) {
-        if (m < a.M) put(a.yb + at, v0);
-        if (m + 1 < a.M) put(a.yb + at + a.ldy, v1);
+        if (m < it.m_end) put(a.yb + at, v0);
+        if (m + 1 < it.m_end) put(a.yb + at + a.ldy, v1);
     } else if (a.accumulate) {
-        if (m < a.M) a.y[at] += v0;
-        if (m + 1 < a.M) a.y[at + a.ldy] += v1;
+        if (m < it.m_end) a.y[at] += v0;
+        if (m + 1 < it.m_end) a.y[at + a.ldy] += v1;
     } else {
-        if (m < a.M) a.y[at] = v0;
-        if (m + 1 < a.M) a.y[at + a.ldy] = v1;
+        if (m < it.m_end) a.y[at] = v0;
+        if (m + 1 < it.m_end) a.y[at + a.ldy] = v1;
     }
 }
 
@@ -166,14 +204,17 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
     __syncthreads();
     tc_fence_after();
     const unsigned tmem = *tmem_slot;
-    FtWalk walk = ft_walk(p);
+    if (p.grouped) pdl_wait();                       // the work list is the previous kernels' result
+    FtWalk walk = ft_walk(a, p);
     bool ok = true;
 
     if (warp == 0) {
         if (lane == 0) {
             // the weight boxes of the first stages do not depend on the previous kernel
             FtWalk ahead = walk;
-            const FtItem first = ft_next(a, p, ahead);
+            const bool any = ft_more(walk);          // a short work list leaves CTAs without a tile
+            FtItem first{};
+            if (any) first = ft_next<TOK>(a, p, ahead);
             auto load_w = [&](uint8_t* st, const FtItem& it, int b, unsigned long long* bar) {
                 if (p.tiled) tma_load_2d(st, &map_w, 0, (it.wt * p.kb + b) * FT_ROWS, bar);
                 else tma_load_2d(st, &map_w, b * FT_KE, it.pl.n0, bar);
@@ -186,8 +227,7 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
             pdl_wait();
             unsigned c = 0;                          // stages issued so far
             while (ft_more(walk) && ok) {
-                const FtItem it = ft_next(a, p, walk);
-                const int row = a.seg_in[it.pl.seg] * p.m_rows + it.tt * TOK;
+                const FtItem it = ft_next<TOK>(a, p, walk);
                 for (int l = 0; l < it.nb; l++, c++) {
                     const int s = c % STAGES;
                     uint8_t* st = stages + (size_t)s * Cfg::STAGE_BYTES;
@@ -197,7 +237,7 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                         mbar_expect_tx(&full[s], Cfg::STAGE_BYTES);
                         load_w(st, it, it.b0 + l, &full[s]);
                     }
-                    tma_load_2d(st + FT_A_BYTES, &map_x, (it.b0 + l) * FT_KE, row, &full[s]);
+                    tma_load_2d(st + FT_A_BYTES, &map_x, (it.b0 + l) * FT_KE, it.x_row, &full[s]);
                 }
             }
             if (!ok) {
@@ -210,7 +250,7 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
         if (lane == 0) {
             unsigned c = 0, t = 0;
             for (; ft_more(walk) && ok; t++) {
-                const FtItem it = ft_next(a, p, walk);
+                const FtItem it = ft_next<TOK>(a, p, walk);
                 const unsigned b = t & 1u;
                 ok = mbar_wait(&tempty[b], ((t >> 1) & 1u) ^ 1u, wl);
                 if (!ok) break;
@@ -236,12 +276,12 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
         unsigned t = 0;
         constexpr size_t PIECE = (size_t)TOK * FT_ROWS;
         for (; ft_more(walk) && ok; t++) {
-            const FtItem it = ft_next(a, p, walk);
+            const FtItem it = ft_next<TOK>(a, p, walk);
             const unsigned b = t & 1u;
             ok = mbar_wait(&tfull[b], (t >> 1) & 1u, wl);
             if (!ok) break;
             tc_fence_after();
-            const int n = it.pl.n0 + q * 32 + lane, m0 = it.tt * TOK + col0;
+            const int n = it.pl.n0 + q * 32 + lane, m0 = it.m0 + col0;
             const unsigned taddr = tmem + ((unsigned)(q * 32) << 16) + b * TOK + col0;
             const bool whole = it.nb == p.kb;
             float* mine = p.part + ((size_t)blockIdx.x * 2 + (it.b0 == 0 ? 1 : 0)) * PIECE + (size_t)col0 * FT_ROWS + q * 32 + lane;
@@ -254,11 +294,11 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                     __syncwarp();
                     if (lane == 0) mbar_arrive(&tempty[b]);
                 }
-                if (m0 + c >= a.M) continue;
+                if (m0 + c >= it.m_end) continue;
                 if (whole) {
 #pragma unroll
                     for (int j = 0; j < 32; j += 2)
-                        ft_emit2(a, it.pl, n, m0 + c + j, __int_as_float(r[j]), __int_as_float(r[j + 1]));
+                        ft_emit2(a, it, n, m0 + c + j, __int_as_float(r[j]), __int_as_float(r[j + 1]));
                 } else {
 #pragma unroll
                     for (int j = 0; j < 32; j++) mine[(size_t)(c + j) * FT_ROWS] = __int_as_float(r[j]);
@@ -288,7 +328,7 @@ k_fgemm_tc(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CU
                         for (int j = 0; j < 32; j++) v[j] += __ldcg(piece + (size_t)j * FT_ROWS);
                     }
 #pragma unroll
-                    for (int j = 0; j < 32; j += 2) ft_emit2(a, it.pl, n, m0 + c + j, v[j], v[j + 1]);
+                    for (int j = 0; j < 32; j += 2) ft_emit2(a, it, n, m0 + c + j, v[j], v[j + 1]);
                 }
             }
             asm volatile("bar.sync 1, %0;" ::"n"(Cfg::EPI_WARPS * 32) : "memory");   // last_cta is read before it is written again
@@ -315,9 +355,38 @@ static CUtensorMap bf16_map(const void* base, size_t rows, int ld, int box_rows)
 }
 
 template <int TOK>
+static void configure() {
+    static bool configured = false;
+    if (configured) return;
+    DETB_CUDA_OK(cudaFuncSetAttribute(k_fgemm_tc<TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)FtCfg<TOK>::SMEM));
+    configured = true;
+}
+// a.M: rows of x
+template <int TOK>
+static void launch_grouped(const FgemmArgs& a, cudaStream_t q) {
+    using Cfg = FtCfg<TOK>;
+    FtPlan p{};
+    p.grouped = 1;
+    p.kb = (a.K + FT_KE - 1) / FT_KE;
+    p.wtiles = (a.group_rows + FT_ROWS - 1) / FT_ROWS;
+    p.tiled = a.wt != nullptr;
+    DETB_REQUIRE(a.ldw == round8(a.K), "linear: weight rows must be padded to 8 elements");
+    const CUtensorMap map_w = p.tiled ? bf16_map(a.wt, (size_t)a.groups * p.wtiles * p.kb * FT_ROWS, FT_KE, FT_ROWS)
+                                      : bf16_map(a.w, a.N, a.ldw, FT_ROWS);
+    const CUtensorMap map_x = bf16_map(a.x, a.M, a.ldx, TOK);
+    configure<TOK>();
+    const int grid = (int)std::min<long long>(sm_count(), (long long)a.max_work * p.wtiles);
+    launch_pdl(k_fgemm_tc<TOK>, dim3(grid), dim3(Cfg::THREADS), Cfg::SMEM, q, 1, map_w, map_x, a, p);
+}
+
+template <int TOK>
 static void launch_tok(FgemmArgs a, cudaStream_t q) {
     using Cfg = FtCfg<TOK>;
     plan_tiles(a, FT_ROWS);
+    if (a.group_rows) {
+        launch_grouped<TOK>(a, q);
+        return;
+    }
     int groups = 1;
     for (int s = 0; s < a.nseg; s++) groups = std::max(groups, a.seg_in[s] + 1);
     FtPlan p{};
@@ -349,11 +418,7 @@ static void launch_tok(FgemmArgs a, cudaStream_t q) {
     p.tiled = a.wt != nullptr;
     const CUtensorMap map_w = p.tiled ? bf16_map(a.wt, (size_t)p.wtiles * p.kb * FT_ROWS, FT_KE, FT_ROWS) : bf16_map(a.w, a.N, a.ldw, FT_ROWS);
     const CUtensorMap map_x = bf16_map(a.x, x_rows, a.ldx, TOK);
-    static bool configured = false;
-    if (!configured) {
-        DETB_CUDA_OK(cudaFuncSetAttribute(k_fgemm_tc<TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM));
-        configured = true;
-    }
+    configure<TOK>();
     launch_pdl(k_fgemm_tc<TOK>, dim3(grid), dim3(Cfg::THREADS), Cfg::SMEM, q, 1, map_w, map_x, a, p);
 }
 
@@ -364,7 +429,13 @@ __global__ void k_flinear_tile(const FgemmArgs a, int kb, bf16* __restrict__ dst
     if (id >= (long long)a.tile0[a.nseg] * per_tile) return;
     const int t = (int)(id / per_tile), i = (int)(id % per_tile);
     const int b = i / (FT_ROWS * 8), r = i / 8 % FT_ROWS, k = b * FT_KE + (i & 7) * 8;
-    const TilePlace pl = place_tile<FT_ROWS>(a, t);
+    TilePlace pl;
+    if (a.group_rows) {
+        const int per = (a.group_rows + FT_ROWS - 1) / FT_ROWS, e = t / per;
+        pl = TilePlace{0, e * a.group_rows + (t - e * per) * FT_ROWS, (e + 1) * a.group_rows};
+    } else {
+        pl = place_tile<FT_ROWS>(a, t);
+    }
     uint4 v = make_uint4(0, 0, 0, 0);
     if (pl.n0 + r < pl.n_end && k < a.ldw) v = *reinterpret_cast<const uint4*>(a.w + (size_t)(pl.n0 + r) * a.ldw + k);
     reinterpret_cast<uint4*>(dst)[id] = v;
@@ -374,6 +445,10 @@ void fgemm_tc_launch(FgemmArgs a, cudaStream_t q) {
     if (a.M <= 32) launch_tok<32>(a, q);
     else if (a.M <= 128) launch_tok<128>(a, q);
     else launch_tok<256>(a, q);
+}
+void fgemm_tc_group_launch(FgemmArgs a, int tok, cudaStream_t q) {
+    if (tok == 32) launch_tok<32>(a, q);
+    else launch_tok<128>(a, q);
 }
 
 }  // namespace detb
@@ -390,6 +465,13 @@ static FgemmArgs tile_args(int K, int nseg, const int* seg_end) {
     return a;
 }
 
+static void tile_rows(const FgemmArgs& a, int nseg, void* dst, cudaStream_t st) {
+    const int kb = (a.K + FT_KE - 1) / FT_KE;
+    const long long n = (long long)a.tile0[nseg] * kb * FT_ROWS * (FT_KE / 8);
+    k_flinear_tile<<<(unsigned)((n + 255) / 256), 256, 0, queue_of(st)>>>(a, kb, static_cast<bf16*>(dst));
+    DETB_CUDA_OK(cudaGetLastError());
+}
+
 extern "C" {
 
 size_t det_f_linear_tile_bytes(int K, int nseg, const int* seg_end) {
@@ -401,10 +483,20 @@ void det_f_linear_tile(const det_flinear* src, int nseg, const int* seg_end, voi
     a.w = static_cast<const bf16*>(src->w);
     a.N = src->N;
     a.ldw = src->ld;
-    const int kb = (src->K + FT_KE - 1) / FT_KE;
-    const long long n = (long long)a.tile0[nseg] * kb * FT_ROWS * (FT_KE / 8);
-    k_flinear_tile<<<(unsigned)((n + 255) / 256), 256, 0, queue_of(st)>>>(a, kb, static_cast<bf16*>(dst));
-    DETB_CUDA_OK(cudaGetLastError());
+    tile_rows(a, nseg, dst, st);
+}
+size_t det_f_linear_tile_groups_bytes(int K, int groups, int rows) {
+    return (size_t)groups * ((rows + FT_ROWS - 1) / FT_ROWS) * ((K + FT_KE - 1) / FT_KE) * FT_A_BYTES;
+}
+void det_f_linear_tile_groups(const det_flinear* src, int groups, void* dst, cudaStream_t st) {
+    DETB_REQUIRE(groups > 0 && src->N % groups == 0 && src->ld % 8 == 0, "linear: bad groups");
+    FgemmArgs a = tile_args(src->K, 1, &src->N);
+    a.group_rows = src->N / groups;
+    a.tile0[1] = groups * ((a.group_rows + FT_ROWS - 1) / FT_ROWS);
+    a.w = static_cast<const bf16*>(src->w);
+    a.N = src->N;
+    a.ldw = src->ld;
+    tile_rows(a, 1, dst, st);
 }
 
 }  // extern "C"

@@ -25,7 +25,8 @@ __device__ __forceinline__ void load_quad(const bf16* const (&row)[R], int k, in
     for (int r = 0; r < R; r++) w[r] = k < kp ? __ldcs(reinterpret_cast<const uint4*>(row[r] + k)) : make_uint4(0, 0, 0, 0);
 }
 
-template <class T, int MT, bool NORM>
+// GROUPED: a quad belongs to a pair (input row, linear of a stack), chosen on the device; xs then holds every input row.
+template <class T, int MT, bool NORM, bool GROUPED = false>
 __global__ void __launch_bounds__(GV_THREADS, 1) k_fgemv(const FgemmArgs a, const GemvPlan p) {
     extern __shared__ __align__(16) float xs[];                     // [ngroups][MT][2 planes][kp / 2]
     __shared__ float red[2][GV_WARPS][GV_ROWS * MT];
@@ -33,7 +34,8 @@ __global__ void __launch_bounds__(GV_THREADS, 1) k_fgemv(const FgemmArgs a, cons
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int ws = p.wsplit, group = warp / ws, part = warp % ws, qpc = GV_WARPS / ws;   // quads per CTA and round
-    const int nquads = a.tile0[a.nseg];
+    const int qpg = GROUPED ? (a.group_rows + GV_ROWS - 1) / GV_ROWS : 0;      // quads of a pair
+    const int nquads = GROUPED ? a.pairs * qpg : a.tile0[a.nseg];
     const int kp = p.kp, half = kp / 2;
     const int stride = qpc * gridDim.x;
     int quad = blockIdx.x * qpc + group;
@@ -41,17 +43,31 @@ __global__ void __launch_bounds__(GV_THREADS, 1) k_fgemv(const FgemmArgs a, cons
     const bf16* row[GV_ROWS];
     uint4 w0[GV_ROWS];
     TilePlace pl{};
+    int pair = 0, n_base = 0;
+    bool none = false;
     auto aim = [&](int t) {
-        pl = place_tile<GV_ROWS>(a, t);
+        if constexpr (GROUPED) {
+            pair = t / qpg;
+            const int e = a.sel[pair];
+            none = e >= a.groups;
+            n_base = (none ? 0 : e) * a.group_rows;
+            pl = TilePlace{pair / a.pairs_per_row, n_base + (t - pair * qpg) * GV_ROWS, n_base + a.group_rows};
+        } else {
+            pl = place_tile<GV_ROWS>(a, t);
+        }
 #pragma unroll
         for (int r = 0; r < GV_ROWS; r++) row[r] = a.w + (size_t)min(pl.n0 + r, pl.n_end - 1) * a.ldw;
     };
     const int kstep = ws * 256, k_first = (part * 32 + lane) * 8;
-    if (quad < nquads) {
+    if (!GROUPED && quad < nquads) {
         aim(quad);
         load_quad(row, k_first, kp, w0);
     }
     pdl_wait();
+    if (GROUPED && quad < nquads) {
+        aim(quad);
+        if (!none) load_quad(row, k_first, kp, w0);
+    }
 
     // ---- stage the input rows
     if constexpr (NORM) {
@@ -85,9 +101,9 @@ __global__ void __launch_bounds__(GV_THREADS, 1) k_fgemv(const FgemmArgs a, cons
 
     int buf = 0;
     for (int base = blockIdx.x * qpc; base < nquads; base += stride, quad += stride, buf ^= 1) {
-        const bool live = quad < nquads;
+        const bool live = quad < nquads && !none;
         if (live) {
-            const float* xg = xs + (size_t)a.seg_in[pl.seg] * MT * kp;
+            const float* xg = xs + (size_t)(GROUPED ? pl.seg : a.seg_in[pl.seg]) * MT * kp;
             float acc[GV_ROWS][MT];
 #pragma unroll
             for (int r = 0; r < GV_ROWS; r++)
@@ -126,10 +142,11 @@ __global__ void __launch_bounds__(GV_THREADS, 1) k_fgemv(const FgemmArgs a, cons
                 }
         }
         const TilePlace here = pl;
+        const int here_pair = pair, here_base = n_base;
         // the next quad's first weights are requested before this one is handed over
         if (quad + stride < nquads) {
             aim(quad + stride);
-            load_quad(row, k_first, kp, w0);
+            if (!none) load_quad(row, k_first, kp, w0);
         }
         if (ws == 1) __syncwarp();
         else if (ws == GV_WARPS) __syncthreads();
@@ -142,8 +159,12 @@ __global__ void __launch_bounds__(GV_THREADS, 1) k_fgemv(const FgemmArgs a, cons
             const float other = __shfl_down_sync(LANES, v, MT);     // row r + 1 of the quad, same m
             if (m < a.M && n < here.n_end) {
                 if (n >= a.glu_from) {
-                    if (!(r & 1)) put(static_cast<T*>(a.h) + (size_t)m * a.ldh + (n - a.glu_from) / 2, silu_fast(v) * other);
+                    if (a.act == DET_FF_RELU2)
+                        put(static_cast<T*>(a.h) + (size_t)(GROUPED ? here_pair : m) * a.ldh + (n - here_base - a.glu_from), relu_squared(v));
+                    else if (!(r & 1))
+                        put(static_cast<T*>(a.h) + (size_t)m * a.ldh + (n - a.glu_from) / 2, gate_pair(a.act, v, other));
                 } else {
+                    if (a.bias) v += a.bias[n];
                     if (a.softcap > 0.0f) v = a.softcap * tanhf(v / a.softcap);
                     const size_t at = (size_t)m * a.ldy + n;
                     if (a.yb) put(a.yb + at, v);
@@ -166,19 +187,19 @@ bool fgemv_takes(const FgemmArgs& a, int) {
     return a.M <= 4 && gemv_smem(a, gemv_mt(a.M)) <= smem_optin() - 8192;
 }
 
-template <class T, int MT, bool NORM>
+template <class T, int MT, bool NORM, bool GROUPED = false>
 static void launch_gemv(const FgemmArgs& a, cudaStream_t q) {
     const size_t smem = gemv_smem(a, MT);
     static size_t configured = 0;
     if (smem > configured) {
-        DETB_CUDA_OK(cudaFuncSetAttribute(k_fgemv<T, MT, NORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        DETB_CUDA_OK(cudaFuncSetAttribute(k_fgemv<T, MT, NORM, GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         configured = smem;
     }
     GemvPlan p;
     p.kp = round8(a.K);
     p.ngroups = (int)(smem / ((size_t)MT * p.kp * sizeof(float)));
     // warps per quad: the smallest split whose last round wastes little; a warp keeps at least one full step of K
-    const int quads = a.tile0[a.nseg], sms = sm_count();
+    const int quads = GROUPED ? a.pairs * ((a.group_rows + GV_ROWS - 1) / GV_ROWS) : a.tile0[a.nseg], sms = sm_count();
     p.wsplit = 1;
     double best = 1e30;
     for (int ws = 1; ws <= GV_WARPS; ws *= 2) {
@@ -192,7 +213,7 @@ static void launch_gemv(const FgemmArgs& a, cudaStream_t q) {
     }
     const int qpc = GV_WARPS / p.wsplit;
     const int grid = std::min(sms, (quads + qpc - 1) / qpc);
-    launch_pdl(k_fgemv<T, MT, NORM>, dim3(grid), dim3(GV_THREADS), smem, q, 1, a, p);
+    launch_pdl(k_fgemv<T, MT, NORM, GROUPED>, dim3(grid), dim3(GV_THREADS), smem, q, 1, a, p);
 }
 
 template <class T, int MT>
@@ -212,6 +233,25 @@ void fgemv_launch(FgemmArgs a, int dtype, cudaStream_t q) {
     plan_tiles(a, GV_ROWS);
     if (dtype == DET_BF16) launch_mt<bf16>(a, q);
     else launch_mt<float>(a, q);
+}
+
+// `rows` input rows become the groups of a one-row call.
+static FgemmArgs group_args(FgemmArgs a, int rows) {
+    a.M = 1;
+    a.nseg = 1;
+    a.seg_end[0] = a.N;
+    a.seg_in[0] = rows - 1;
+    a.gstride = a.ldx;
+    return a;
+}
+bool fgemv_group_takes(const FgemmArgs& a, int rows) {
+    if (float_flags() & 2) return false;
+    return rows <= 4 && gemv_smem(group_args(a, rows), 1) <= smem_optin() - 8192;
+}
+void fgemv_group_launch(FgemmArgs a, int dtype, cudaStream_t q) {
+    a = group_args(a, a.pairs / a.pairs_per_row);
+    if (dtype == DET_BF16) launch_gemv<bf16, 1, false, true>(a, q);
+    else launch_gemv<float, 1, false, true>(a, q);
 }
 
 }  // namespace detb

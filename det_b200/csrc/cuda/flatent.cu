@@ -7,7 +7,7 @@
 //     keys staged in shared memory, online softmax; k_latent_out merges the ranges, adds the sink, applies W_uv and the gate.
 //   expanded (a run of tokens with bfloat16 activations): keys and values of the cached rows are multiplied out by the
 //     tensor-core GEMM, then k_latent_flash computes 64 query rows of a head against 64-key tiles with bfloat16 MMAs.
-#include "fops.cuh"
+#include "flash.cuh"
 #include <algorithm>
 #include <cmath>
 #include <type_traits>
@@ -44,7 +44,6 @@ struct LatentArgs {
     det_seq_ref seq;
 };
 
-__device__ __forceinline__ int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
 // element e of the rotated part of a head at `pos` (pairs (2i, 2i + 1) of the first rot_dims elements)
 __device__ __forceinline__ float rotated(const float* x, int e, int pos, const LatentArgs& a) {
     if (e >= a.rot_dims) return x[e];
@@ -322,238 +321,54 @@ __global__ void __launch_bounds__(256) k_latent_out(const LatentArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------------------ expanded form
-constexpr int FL_ROWS = 64, FL_KEYS = 64, FL_WARPS = 4;
-
-__device__ __forceinline__ void ldsm4(unsigned addr, unsigned (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldsm4_t(unsigned addr, unsigned (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void mma16816(float (&d)[4], const unsigned (&a)[4], unsigned b0, unsigned b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-// 2^x by the special function unit (relative error about 2^-22; 2^-inf = 0).
-__device__ __forceinline__ float exp2_fast(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
+// One head of the expanded form for the flash loop: keys are [expanded part | rotated part of the cache row].
+struct LatentFlash {
+    const LatentArgs& a;
+    int h;
+    const bf16* cache;
+    __device__ __forceinline__ LatentFlash(const LatentArgs& args, int head)
+        : a(args), h(head), cache(static_cast<const bf16*>(args.seq.one.cache)) {}
+    __device__ __forceinline__ unsigned query(int row, int pos, int e) const {
+        if (e >= a.dim + a.rot_dim) return 0;                      // dim and rot_dim are multiples of 8: pairs do not straddle
+        const float* q = a.q + (size_t)row * a.ldq + h * (a.dim + a.rot_dim);
+        const float qs = a.scale * 1.4426950408889634f;            // scores in units of log 2
+        float u = q[e], v = q[e + 1];
+        const int er = e - a.dim;
+        if (er >= 0 && er < a.rot_dims) {
+            const size_t at = (size_t)pos * (a.rot_dims / 2) + (er >> 1);
+            const float c = a.rope_cos[at], s = a.rope_sin[at], x = u;
+            u = fmaf(x, c, -(v * s));
+            v = fmaf(v, c, x * s);
+        }
+        return pack_bf(u * qs, v * qs);
+    }
+    __device__ __forceinline__ int pieces() const { return (a.dim + a.rot_dim + a.vdim) / 8; }
+    __device__ __forceinline__ FlashPiece piece(int v) const {
+        const int kvec = a.dim / 8, rvec = a.rot_dim / 8;
+        if (v < kvec) return {a.kv + h * a.dim + v * 8, a.ldkv, v, false};
+        if (v < kvec + rvec) return {cache + a.rp + (v - kvec) * 8, a.ld, v, false};
+        return {a.kv + a.heads * a.dim + h * a.vdim + (v - kvec - rvec) * 8, a.ldkv, v - kvec - rvec, true};
+    }
+    __device__ __forceinline__ float inverse(float m, float l) const {
+        if (!a.sink) return 1.0f / l;
+        const float s2 = a.sink[h] * 1.4426950408889634f, top = fmaxf(m, s2), e = exp2f(m - top);
+        return e / (l * e + exp2f(s2 - top));
+    }
+    __device__ __forceinline__ void store(int row, int, int v, float o0, float o1) const {
+        if (v >= a.vdim) return;
+        const float* gate = a.y + (size_t)row * a.ldy + a.gate_off + h * a.vdim;
+        bf16* out = static_cast<bf16*>(a.out) + (size_t)row * a.ldo + h * a.vdim;
+        *reinterpret_cast<unsigned*>(out + v) = pack_bf(o0 * sigmoid_fast(gate[v]), o1 * sigmoid_fast(gate[v + 1]));
+    }
+};
 
 // One head x 64 query rows; DV = value dimensions rounded up to a multiple of 64.
 template <int DV>
 __global__ void __launch_bounds__(FL_WARPS * 32, 2) k_latent_flash(const LatentArgs a) {
-    extern __shared__ __align__(16) uint8_t fsm[];
-    const int hd = a.dim + a.rot_dim, dqp = (hd + 15) & ~15, ldk = dqp + 8;
-    constexpr int LDV = DV + 8;
-    bf16* Q = reinterpret_cast<bf16*>(fsm);                       // [64][ldk]
-    bf16* Kt = Q + FL_ROWS * ldk;                                  // [2][64][ldk]
-    bf16* Vt = Kt + 2 * FL_KEYS * ldk;                             // [2][64][LDV]
-    const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    // later query rows have more keys behind them (until the window fills): start those first
-    const int r0 = (gridDim.x - 1 - blockIdx.x) * FL_ROWS, nrows = min(FL_ROWS, a.M - r0);
-    constexpr int NT = FL_WARPS * 32;
-    pdl_trigger();
-    for (int i = threadIdx.x; i < (2 * FL_KEYS * ldk + 2 * FL_KEYS * LDV) / 8; i += NT)
-        reinterpret_cast<uint4*>(Kt)[i] = make_uint4(0, 0, 0, 0);
-    pdl_wait();
-    const int p0 = position_of(a.seq, r0), p_last = p0 + nrows - 1;
-    const float qs = a.scale * 1.4426950408889634f;                // scores in units of log 2
-#pragma unroll 4
-    for (int r = warp; r < FL_ROWS; r += FL_WARPS) {               // a warp per row, two neighbouring elements per lane
-        const float* q = a.q + (size_t)(r0 + min(r, nrows - 1)) * a.ldq + h * hd;
-        for (int e = lane * 2; e < dqp; e += 64) {
-            float u = 0.0f, v = 0.0f;
-            if (r < nrows && e < hd) {                             // dim and rot_dim are multiples of 8: pairs do not straddle
-                u = q[e];
-                v = q[e + 1];
-                const int er = e - a.dim;
-                if (er >= 0 && er < a.rot_dims) {
-                    const size_t at = (size_t)(p0 + r) * (a.rot_dims / 2) + (er >> 1);
-                    const float c = a.rope_cos[at], s = a.rope_sin[at], x = u;
-                    u = fmaf(x, c, -(v * s));
-                    v = fmaf(v, c, x * s);
-                }
-            }
-            *reinterpret_cast<unsigned*>(Q + r * ldk + e) = pack_bf(u * qs, v * qs);
-        }
-    }
-    const bf16* cache = static_cast<const bf16*>(a.seq.one.cache);
-    const int kvec = a.dim / 8, rvec = a.rot_dim / 8, vvec = a.vdim / 8, tvec = kvec + rvec + vvec;
-    // a warp copies whole key rows; which 16-byte pieces of a row a lane takes does not depend on the row
-    constexpr int PIECES = 3;
-    const bf16* piece[PIECES];
-    int step[PIECES];
-    unsigned to[PIECES], ldt[PIECES];
-#pragma unroll
-    for (int j = 0; j < PIECES; j++) {
-        const int v = lane + j * 32;
-        piece[j] = nullptr;
-        step[j] = a.ldkv;
-        to[j] = 0;
-        ldt[j] = ldk * 2;
-        if (v < kvec) {
-            piece[j] = a.kv + h * a.dim + v * 8;
-            to[j] = smem_addr(Kt + v * 8);
-        } else if (v < kvec + rvec) {
-            piece[j] = cache + a.rp + (v - kvec) * 8;
-            step[j] = a.ld;
-            to[j] = smem_addr(Kt + v * 8);
-        } else if (v < tvec) {
-            piece[j] = a.kv + a.heads * a.dim + h * a.vdim + (v - kvec - rvec) * 8;
-            to[j] = smem_addr(Vt + (v - kvec - rvec) * 8);
-            ldt[j] = LDV * 2;
-        }
-    }
-    auto fetch = [&](int k0, int buf) {
-        const int slot0 = k0 % a.cap, last = p_last - k0;         // past the last key: a copy of it, masked below
-#pragma unroll
-        for (int j = 0; j < PIECES; j++) {
-            if (!piece[j]) continue;
-            unsigned dst = to[j] + (unsigned)(buf * FL_KEYS + warp) * ldt[j];
-#pragma unroll 4
-            for (int k = warp; k < FL_KEYS; k += FL_WARPS, dst += FL_WARPS * ldt[j]) {
-                int slot = slot0 + min(k, last);
-                if (slot >= a.cap) slot = a.cap >= FL_KEYS ? slot - a.cap : slot % a.cap;
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(piece[j] + (long long)slot * step[j]) : "memory");
-            }
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    __syncthreads();
-    float o[DV / 8][4];
-#pragma unroll
-    for (int i = 0; i < DV / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
-    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
-    const int pa = p0 + warp * 16 + (lane >> 2), pb = pa + 8;       // positions of this lane's two rows
-    const int lo = first_key(p0, a.window);
-    const unsigned qaddr = smem_addr(Q + (warp * 16 + (lane & 15)) * ldk + (lane >> 4) * 8);
-    int buf = 0;
-    fetch(lo, 0);
-    for (int k0 = lo; k0 <= p_last; k0 += FL_KEYS, buf ^= 1) {
-        if (k0 + FL_KEYS <= p_last) {
-            fetch(k0 + FL_KEYS, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        // keys of this tile that some row of the warp sees
-        const int w_first = p0 + warp * 16, w_last = w_first + 15;
-        const bool seen = k0 <= w_last && (a.window <= 0 || k0 + FL_KEYS - 1 > w_first - a.window);
-        if (seen) {
-            float s[8][4];
-#pragma unroll
-            for (int i = 0; i < 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
-            const bf16* K = Kt + (size_t)buf * FL_KEYS * ldk;
-            const unsigned kaddr = smem_addr(K + ((lane & 7) + ((lane >> 4) << 3)) * ldk + ((lane >> 3) & 1) * 8);
-#pragma unroll 2
-            for (int kk = 0; kk < dqp; kk += 16) {
-                unsigned qa[4];
-                ldsm4(qaddr + kk * 2, qa);
-#pragma unroll
-                for (int n = 0; n < 4; n++) {
-                    unsigned kb[4];
-                    ldsm4(kaddr + (unsigned)(n * 16 * ldk + kk) * 2, kb);
-                    mma16816(s[2 * n], qa, kb[0], kb[1]);
-                    mma16816(s[2 * n + 1], qa, kb[2], kb[3]);
-                }
-            }
-            const bool edge = k0 + FL_KEYS - 1 > w_first || (a.window > 0 && k0 <= w_last - a.window);
-            if (edge) {
-#pragma unroll
-                for (int n = 0; n < 8; n++)
-#pragma unroll
-                    for (int c = 0; c < 4; c++) {
-                        const int j = k0 + n * 8 + (lane & 3) * 2 + (c & 1), p = c < 2 ? pa : pb;
-                        if (j > p || (a.window > 0 && j <= p - a.window)) s[n][c] = -INFINITY;
-                    }
-            }
-            float mx[2] = {m[0], m[1]};
-#pragma unroll
-            for (int n = 0; n < 8; n++) {
-                mx[0] = fmaxf(mx[0], fmaxf(s[n][0], s[n][1]));
-                mx[1] = fmaxf(mx[1], fmaxf(s[n][2], s[n][3]));
-            }
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                mx[i] = fmaxf(mx[i], __shfl_xor_sync(FULL, mx[i], 1));
-                mx[i] = fmaxf(mx[i], __shfl_xor_sync(FULL, mx[i], 2));
-            }
-            float f[2], base[2];
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                base[i] = mx[i] == -INFINITY ? 0.0f : mx[i];       // no key seen yet: every weight below is exp2(-inf) = 0
-                f[i] = exp2_fast(m[i] - base[i]);
-                m[i] = mx[i];
-                l[i] *= f[i];
-            }
-            if (__any_sync(FULL, f[0] != 1.0f || f[1] != 1.0f)) {
-#pragma unroll
-                for (int i = 0; i < DV / 8; i++) {
-                    o[i][0] *= f[0];
-                    o[i][1] *= f[0];
-                    o[i][2] *= f[1];
-                    o[i][3] *= f[1];
-                }
-            }
-            unsigned pf[4][4];
-#pragma unroll
-            for (int n = 0; n < 8; n++) {
-                const float e0 = exp2_fast(s[n][0] - base[0]), e1 = exp2_fast(s[n][1] - base[0]);
-                const float e2 = exp2_fast(s[n][2] - base[1]), e3 = exp2_fast(s[n][3] - base[1]);
-                l[0] += e0 + e1;
-                l[1] += e2 + e3;
-                pf[n >> 1][(n & 1) * 2] = pack_bf(e0, e1);
-                pf[n >> 1][(n & 1) * 2 + 1] = pack_bf(e2, e3);
-            }
-            const bf16* V = Vt + (size_t)buf * FL_KEYS * LDV;
-            const unsigned vaddr = smem_addr(V + (lane & 15) * LDV + (lane >> 4) * 8);
-#pragma unroll
-            for (int kk = 0; kk < 4; kk++)
-#pragma unroll
-                for (int n = 0; n < DV / 16; n++) {
-                    unsigned vb[4];
-                    ldsm4_t(vaddr + (unsigned)(kk * 16 * LDV + n * 16) * 2, vb);
-                    mma16816(o[2 * n], pf[kk], vb[0], vb[1]);
-                    mma16816(o[2 * n + 1], pf[kk], vb[2], vb[3]);
-                }
-        }
-        __syncthreads();
-    }
-#pragma unroll
-    for (int i = 0; i < 2; i++) {
-        l[i] += __shfl_xor_sync(FULL, l[i], 1);
-        l[i] += __shfl_xor_sync(FULL, l[i], 2);
-        const int r = warp * 16 + (lane >> 2) + i * 8;
-        if (r >= nrows) continue;
-        float scale_o = 1.0f / l[i];
-        if (a.sink) {
-            const float s2 = a.sink[h] * 1.4426950408889634f, top = fmaxf(m[i], s2), e = exp2f(m[i] - top);
-            scale_o = e / (l[i] * e + exp2f(s2 - top));
-        }
-        const float* gate = a.y + (size_t)(r0 + r) * a.ldy + a.gate_off + h * a.vdim;
-        bf16* out = static_cast<bf16*>(a.out) + (size_t)(r0 + r) * a.ldo + h * a.vdim;
-#pragma unroll
-        for (int n = 0; n < DV / 8; n++) {
-            const int v = n * 8 + (lane & 3) * 2;
-            if (v < a.vdim)
-                *reinterpret_cast<unsigned*>(out + v) = pack_bf(o[n][i * 2] * scale_o * sigmoid_fast(gate[v]),
-                                                                o[n][i * 2 + 1] * scale_o * sigmoid_fast(gate[v + 1]));
-        }
-    }
+    flash_tile<DV>(LatentFlash(a, blockIdx.y), FlashShape{a.dim + a.rot_dim, a.window, a.cap, a.M}, a.seq);
 }
 
 // ------------------------------------------------------------------------------------------------------ host side
-static size_t flash_smem(int hd, int dv) {
-    const int ldk = ((hd + 15) & ~15) + 8;
-    return ((size_t)(FL_ROWS + 2 * FL_KEYS) * ldk + 2 * (size_t)FL_KEYS * (dv + 8)) * 2;
-}
 // Runs of at least 32 tokens of one sequence with bfloat16 activations and head sizes in whole 16-byte pieces.
 static bool takes_flash(int M, bool one_seq, int dtype, int heads, int dim, int rot_dim, int vdim) {
     return one_seq && dtype == DET_BF16 && M >= 32 && !(float_flags() & 8) && dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 &&

@@ -23,6 +23,12 @@ __device__ __forceinline__ unsigned pack_bf(float lo, float hi) {
 
 __device__ __forceinline__ float sigmoid_fast(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_fast(float z) { return z / (1.0f + expf(-z)); }
+// first half of a feed-forward (DET_FF_*)
+__device__ __forceinline__ float gate_pair(int act, float g, float u) { return (act == DET_FF_REGLU ? fmaxf(g, 0.0f) : silu_fast(g)) * u; }
+__device__ __forceinline__ float relu_squared(float v) {
+    const float r = fmaxf(v, 0.0f);
+    return r * r;
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -73,7 +79,16 @@ struct FgemmArgs {
     float softcap;
     void* h;
     int ldh;
+    const float* bias;       // of rows before glu_from, or NULL
+    int act;
     int* error_flag;
+    // Stacked linears (one per expert, group_rows rows each): which rows meet which linear is known on the device only.
+    int group_rows;          // 0: one linear
+    const int* sel;          // GEMV: linear of pair p, whose input is row p / pairs_per_row; >= groups: none
+    int groups, pairs, pairs_per_row;
+    const int4* work;        // GEMM: {linear, first row, row after the last, -} per token tile
+    const int* nwork;
+    int max_work;
 };
 // Segment of tile `t` and the first weight row of the tile (tiles of ROWS rows never straddle a segment).
 struct TilePlace {
@@ -103,6 +118,13 @@ bool fgemv_takes(const FgemmArgs& a, int dtype);                         // fgem
 void fgemv_launch(FgemmArgs a, int dtype, cudaStream_t q);
 void fgemm_tc_launch(FgemmArgs a, cudaStream_t q);                       // fgemm_tc.cu (bfloat16 activations)
 void fgemm_simt_launch(FgemmArgs a, cudaStream_t q);                     // fgemm.cu (fp32 activations)
+// The same over stacked linears; `a` carries group_rows and sel (GEMV) or work (GEMM).  Tiles of a work list have
+// fgemm_group_tok(dtype, rows per linear) tokens.
+bool fgemv_group_takes(const FgemmArgs& a, int rows);
+void fgemv_group_launch(FgemmArgs a, int dtype, cudaStream_t q);
+int fgemm_group_tok(int dtype, int rows);
+void fgemm_group_launch(FgemmArgs a, int dtype, int tok, cudaStream_t q);
+void fgemm_tc_group_launch(FgemmArgs a, int tok, cudaStream_t q);
 // z[M][N] = f(W act(x) + bias), all in 32-bit (the decay of a linear recurrence)
 void fdecay_launch(const det_flinear* w2, const float* low, int ldlow, const float* bias, int kind, float tau, int M, float* z,
                    cudaStream_t q);

@@ -135,13 +135,14 @@ struct FLinear {
     Buf<uint16_t> w;
     size_t n = 0, k = 0, ld = 0;
     std::vector<int> seg_end;   // rows in segments of their own inputs (det_fgemm_op)
+    size_t groups = 0;          // > 0: a stack of that many equally large linears (det_fmoe_op)
     Buf<uint16_t> tiles;        // backend's second copy for batches, may be empty (Backend::f_linear_ready)
     det_flinear view() const { return det_flinear{w.ptr(), (int)n, (int)k, (int)ld, tiles.ptr()}; }
 };
-// What one sequence keeps in one layer; a layer uses the members it needs.
+// What one sequence keeps in one layer run; a layer uses the members it needs.
 struct FloatState {
-    Buf<float> s;          // recurrent state [heads][dk][dv]
-    Buf<float> prev;       // the previous token's normalised row
+    Buf<float> s;          // recurrent state [heads][dk][dv], or [channels]
+    Buf<float> prev;       // normalised rows of the latest tokens (token shift: one, a convolution: taps - 1)
     Buf<uint8_t> cache;    // `cap` cache rows, used as a ring
     size_t cap = 0;
 };
@@ -253,6 +254,10 @@ class Backend {
     virtual void f_recur(const det_frecur_op&) { no_float_ops(); }             // the backend supplies `scratch`
     virtual void f_latent_prep(const det_flatent_op&) { no_float_ops(); }
     virtual void f_latent_attn(const det_flatent_op&, size_t) { no_float_ops(); }   // supplies `scratch`; bound on any position
+    virtual void f_seam(const det_fseam_op&) { no_float_ops(); }
+    virtual void f_attn(const det_fattn_op&) { no_float_ops(); }   // both steps of det_fattn_op; supplies `scratch`
+    virtual void f_mingru(const det_fmingru_op&) { no_float_ops(); }
+    virtual void f_moe(const det_fmoe_op&, size_t) { no_float_ops(); }   // supplies `scratch` and `counts`; bound on any call's rows
     virtual int32_t argmax(const Buf<float>& logits, size_t v) = 0;
     virtual int32_t sample(const Buf<float>& logits, size_t v, float inv_temp, size_t top_k, float top_p,
                            uint64_t z) = 0;

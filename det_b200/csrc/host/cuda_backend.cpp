@@ -580,6 +580,11 @@ void CudaBackend::f_linear_ready(FLinear& l) {
     if (!int8_layout) return;
     const int nseg = (int)l.seg_end.size();
     const det_flinear src = l.view();
+    if (l.groups) {
+        l.tiles = alloc<uint16_t>(det_f_linear_tile_groups_bytes((int)l.k, (int)l.groups, (int)(l.n / l.groups)) / 2);
+        det_f_linear_tile_groups(&src, (int)l.groups, l.tiles.ptr(), ST);
+        return;
+    }
     l.tiles = alloc<uint16_t>(det_f_linear_tile_bytes((int)l.k, nseg, l.seg_end.data()) / 2);
     det_f_linear_tile(&src, nseg, l.seg_end.data(), l.tiles.ptr(), ST);
 }
@@ -608,6 +613,31 @@ void CudaBackend::f_latent_attn(const det_flatent_op& op_, size_t max_ctx) {
     op.scratch = scratch(float_scratch_, det_f_latent_scratch_bytes(op.M, op.heads, op.dim, op.rot_dim, op.vdim, op.kv_rank, op.window,
                                                                     op.cap, (int)max_ctx - 1, op.dtype));
     det_f_latent_attn(&op, ST);
+}
+
+void CudaBackend::f_seam(const det_fseam_op& op) {
+    flush_pending();
+    det_f_seam(&op, ST);
+}
+void CudaBackend::f_attn(const det_fattn_op& op_) {
+    flush_pending();
+    det_fattn_op op = op_;
+    if (pos_dev && !op.seq.table) op.max_pos = std::min(max_pos, op.cap - 1);
+    op.scratch = scratch(float_scratch_, det_f_attn_scratch_bytes(op.vdim));
+    det_f_attn_prep(&op, ST);
+    det_f_attn(&op, ST);
+}
+void CudaBackend::f_mingru(const det_fmingru_op& op) {
+    flush_pending();
+    det_f_mingru(&op, ST);
+}
+void CudaBackend::f_moe(const det_fmoe_op& op_, size_t max_rows) {
+    flush_pending();
+    det_fmoe_op op = op_;
+    if (moe_counts_.len() < DET_MAX_ROUTER + 1) moe_counts_ = alloc<uint32_t>(DET_MAX_ROUTER + 1);   // zero-filled
+    op.counts = moe_counts_.ptr();
+    op.scratch = scratch(float_scratch_, det_f_moe_scratch_bytes((int)max_rows, op.experts, op.top, op.ff, op.n, op.dtype));
+    det_f_moe(&op, ST);
 }
 
 // cuda.rs:425-471

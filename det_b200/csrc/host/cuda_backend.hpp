@@ -66,6 +66,10 @@ class CudaBackend : public Backend {
     void f_recur(const det_frecur_op& op) override;
     void f_latent_prep(const det_flatent_op& op) override;
     void f_latent_attn(const det_flatent_op& op, size_t max_ctx) override;
+    void f_seam(const det_fseam_op& op) override;
+    void f_attn(const det_fattn_op& op) override;
+    void f_mingru(const det_fmingru_op& op) override;
+    void f_moe(const det_fmoe_op& op, size_t max_rows) override;
     int32_t argmax(const Buf<float>& logits, size_t v) override;
     int32_t sample(const Buf<float>& logits, size_t v, float inv_temp, size_t top_k, float top_p, uint64_t z) override;
 
@@ -144,6 +148,7 @@ class CudaBackend : public Backend {
     void* scratch(Buf<uint8_t>& slot, size_t bytes);
     void finish_linear(CudaLinear& l);
     Buf<uint8_t> attn_scratch_, gdn_scratch_, sample_scratch_, synth_scratch_, float_scratch_;
+    Buf<uint32_t> moe_counts_;       // zero between calls
     Buf<float> swiglu_h_;            // SwiGLU product of a fused gate|up GEMV (the next GEMV quantizes it in its prologue)
     Buf<uint32_t> swiglu_amax_;      // its group maxima, folded by that GEMV's epilogue and consumed by the next one's prologue
     Buf<int32_t> pick_, picks_;

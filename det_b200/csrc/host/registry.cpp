@@ -21,6 +21,10 @@ static Json read_config(const std::string& dir) {
     }
 }
 
+static std::unique_ptr<Model> open_hybrid(const std::string& path, Backend* bk, const OpenOptions& o) {
+    return HybridModel::load_dir(path, read_config(path), bk, o.max_ctx, o.max_batch, o.dtype);
+}
+
 const std::vector<Architecture>& architectures() {
     static const std::vector<Architecture> table = {
         {"qwen35", false,
@@ -30,10 +34,8 @@ const std::vector<Architecture>& architectures() {
              if (!m) throw std::runtime_error(err);
              return m;
          }},
-        {"Fazilorn", true,
-         [](const std::string& path, Backend* bk, const OpenOptions& o) -> std::unique_ptr<Model> {
-             return HybridModel::load_dir(path, read_config(path), bk, o.max_ctx, o.max_batch, o.dtype);
-         }},
+        {"Fazilorn", true, open_hybrid},
+        {"Dopipel", true, open_hybrid},
     };
     return table;
 }

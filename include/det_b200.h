@@ -397,6 +397,9 @@ typedef struct {
 } det_flinear;
 size_t det_f_linear_tile_bytes(int K, int nseg, const int* seg_end);
 void det_f_linear_tile(const det_flinear* src, int nseg, const int* seg_end, void* dst, cudaStream_t st);
+/* The same for a stack of `groups` equally large linears (the experts of a mixture): N = groups * rows. */
+size_t det_f_linear_tile_groups_bytes(int K, int groups, int rows);
+void det_f_linear_tile_groups(const det_flinear* src, int groups, void* dst, cudaStream_t st);
 
 /* What one sequence keeps in one layer: recurrent state s[heads][dk][dv], the previous token's normalised row prev[n], and
  * a cache of `cap` rows used as a ring (the row of position p is row p % cap).  A layer uses the members it needs.     */
@@ -439,10 +442,14 @@ void det_f_norm(const det_fnorm_op* op, cudaStream_t st);
  *     (x + seg_in[i] * group_stride elements), so that linears over different inputs go out as one launch;
  *   - norm_x != NULL (one group only): the input rows are the RMS norm of norm_x (norm_w, eps).  A decode-sized call
  *     builds them in its prologue; a larger one runs det_f_norm into x first (x is then written);
- *   - rows of W from glu_from on (a segment start, or N for none) are (gate, up) pairs: h[row][(n - glu_from) / 2] =
- *     silu(gate) * up, in the activation type;
- *   - rows before glu_from land in y[row][n] (fp32, or bfloat16 with y_bf16), added to it with `accumulate`;
- *     softcap > 0: softcap * tanh(y / softcap).                                                                        */
+ *   - rows of W from glu_from on (a segment start, or N for none) are the first half of a feed-forward and land in h in the
+ *     activation type.  act DET_FF_SWIGLU, DET_FF_REGLU: (gate, up) pairs, h[row][(n - glu_from) / 2] = silu(gate) * up or
+ *     max(gate, 0) * up; DET_FF_RELU2: single rows, h[row][n - glu_from] = max(v, 0)^2;
+ *   - rows before glu_from land in y[row][n] (fp32, or bfloat16 with y_bf16), bias[n] (fp32, NULL: none) added; added to
+ *     what is there with `accumulate`; softcap > 0: softcap * tanh(y / softcap).                                        */
+#define DET_FF_SWIGLU 0
+#define DET_FF_REGLU 1
+#define DET_FF_RELU2 2
 typedef struct {
     const det_flinear* lin;
     int dtype;
@@ -464,6 +471,8 @@ typedef struct {
     float softcap;
     void* h;
     int ldh;
+    const float* bias;
+    int act;
 } det_fgemm_op;
 void det_f_gemm(const det_fgemm_op* op, cudaStream_t st);
 
@@ -542,6 +551,113 @@ size_t det_f_latent_scratch_bytes(int M, int heads, int dim, int rot_dim, int vd
                                   int dtype);
 void det_f_latent_prep(const det_flatent_op* op, cudaStream_t st);
 void det_f_latent_attn(const det_flatent_op* op, cudaStream_t st);
+
+/* The seam between two sublayers of a decoder that normalises both ends of a sublayer, on residual rows x[M][n] (fp32):
+ *   y != NULL:  x += y / sqrt(mean(y^2) + eps) * y_norm * y_scale     (y_scale NULL: 1; y is fp32 with row stride ldy)
+ *   h = x / sqrt(mean(x^2) + eps) * w                                  (w NULL: h = x)
+ *   conv != NULL: h_t += sum_j conv[j] * h_(t - taps + 1 + j) per channel (conv [taps][n], 2 <= taps <= DET_MAX_TAPS), the
+ *                earlier rows coming from the sequence's prev [taps - 1][n], oldest first, which then holds the latest ones
+ *   out[row][.] = h in the activation type (out NULL: only x is updated)
+ * `rstd` [M] is scratch, needed with conv over several tokens of one sequence.                                         */
+#define DET_MAX_TAPS 16
+typedef struct {
+    float* x;
+    int M, n;
+    float eps;
+    const float* y;
+    int ldy;
+    const float* y_norm;
+    const float* y_scale;
+    const float* w;
+    const float* conv;
+    int taps;
+    float* rstd;
+    int dtype;
+    void* out;
+    int ld;
+    det_seq_ref seq;          /* only with conv */
+} det_fseam_op;
+void det_f_seam(const det_fseam_op* op, cudaStream_t st);
+
+/* Attention over grouped key/value heads.  Inputs are columns of the fp32 rows y (stride ldy): q [heads * dim],
+ * k [kv_heads * dim], v [kv_heads * vdim], gate [heads] (gate_off < 0: none).  Query head h reads key/value head
+ * h / (heads / kv_heads).  q and k are rotated in their first rot_dims dimensions, pairs (2i, 2i + 1) (tables
+ * [position][rot_dims / 2]); with vrope_cos / vrope_sin ([position][vdim / 2]) values are rotated too, over all of vdim, and
+ * a head's output is turned back by the query's position.  A cache row holds the rotated keys and values of one position in
+ * the activation type (det_f_attn_ld elements: every head's key and value padded to a multiple of 8).
+ * det_f_attn_prep writes the rows' cache entries and the scaled rotated queries q (activation type, det_f_attn_q_ld elements
+ * a row); det_f_attn: softmax(scale * q . k) over the positions j <= i, out[row][head * vdim + j] = value * sigmoid(gate).
+ * max_pos bounds the positions; the caller guarantees cap > max_pos.                                                   */
+typedef struct {
+    int heads, kv_heads, dim, vdim, rot_dims;
+    float scale;
+    int cap;
+    int M;
+    int dtype;
+    const float* y;
+    int ldy;
+    int q_off, k_off, v_off, gate_off;
+    const float* rope_cos;
+    const float* rope_sin;
+    const float* vrope_cos;
+    const float* vrope_sin;
+    void* q;
+    void* out;
+    int ldo;
+    int max_pos;
+    void* scratch;
+    det_seq_ref seq;
+} det_fattn_op;
+int det_f_attn_ld(int kv_heads, int dim, int vdim);
+int det_f_attn_q_ld(int heads, int dim);
+size_t det_f_attn_scratch_bytes(int vdim);
+void det_f_attn_prep(const det_fattn_op* op, cudaStream_t st);
+void det_f_attn(const det_fattn_op* op, cudaStream_t st);
+
+/* Minimal gated recurrence over n channels: z = sigmoid(y[z_off]), u = y[x_off], candidate = u >= 0 ? u + 1/2 : sigmoid(u),
+ * S <- (1 - z) S + z * candidate, out = S * silu(y[gate_off]) in the activation type.  S is s[n] of the sequence.       */
+typedef struct {
+    int n;
+    int M;
+    int dtype;
+    const float* y;
+    int ldy;
+    int z_off, x_off, gate_off;
+    void* out;
+    int ldo;
+    det_seq_ref seq;
+} det_fmingru_op;
+void det_f_mingru(const det_fmingru_op* op, cudaStream_t st);
+
+/* A mixture of experts over the rows x (activation type, stride ldx, n columns).  z[row][experts + identity] are the router's
+ * logits (fp32, stride ldz).  s = softmax(z); the `top` largest of s + correction are chosen, weighted by s / (sum of the
+ * chosen s + 1e-20).  Expert e: W_down[e] max(W_up[e] x, 0)^2, `up` holding the experts' rows [experts * ff], `down`
+ * [experts * n]; an output from `experts` on is x itself.  shared (NULL: none): its first half hs[row][shared->K] (activation
+ * type, stride ldhs) goes through this linear and is added, times sigmoid of the logit at column shared_gate of z (< 0: 1).
+ * out[row][n] fp32, stride ldo.  `counts` (experts + 1 words) is zero between calls.                                   */
+typedef struct {
+    int experts, identity, top, ff, n;
+    int M;
+    int dtype;
+    const float* z;
+    int ldz;
+    const float* correction;  /* [experts + identity] or NULL */
+    const void* x;
+    int ldx;
+    const det_flinear* up;
+    const det_flinear* down;
+    const det_flinear* shared;
+    const void* hs;
+    int ldhs;
+    int shared_gate;
+    float* out;
+    int ldo;
+    unsigned* counts;
+    void* scratch;
+} det_fmoe_op;
+#define DET_MAX_ROUTER 1024
+size_t det_f_moe_scratch_bytes(int M, int experts, int top, int ff, int n, int dtype);
+void det_f_moe(const det_fmoe_op* op, cudaStream_t st);
 
 /* Measurement switches of the floating-point ops (results agree up to rounding): bit 0 no norm in the GEMV's prologue, bit 1 no
  * GEMV, bit 2 no split of K in the tensor-core GEMM, bit 3 no tensor-core attention.                                   */

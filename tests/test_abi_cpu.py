@@ -77,7 +77,9 @@ def test_ctypes_mirror_has_the_layout_the_c_compiler_gives_the_header(libs, tmp_
              "det_gdn_layer": libs.GdnLayer, "det_gdn_state": libs.GdnState, "det_act_source": libs.ActSource,
              "det_gemv_op": libs.GemvOp, "det_flinear": libs.FLinear, "det_seq_slot": libs.SeqSlot,
              "det_seq_ref": libs.SeqRef, "det_fnorm_op": libs.FNormOp, "det_fgemm_op": libs.FGemmOp,
-             "det_frecur_op": libs.FRecurOp, "det_flatent_op": libs.FLatentOp}
+             "det_frecur_op": libs.FRecurOp, "det_flatent_op": libs.FLatentOp,
+             "det_fseam_op": libs.FSeamOp, "det_fattn_op": libs.FAttnOp, "det_fmingru_op": libs.FMinGruOp,
+             "det_fmoe_op": libs.FMoeOp}
     lines = ['#include <stdio.h>', '#include <stddef.h>', '#include "det_b200.h"', "int main(void) {"]
     for cname, mirror in pairs.items():
         lines.append(f'  printf("{cname} %zu\\n", sizeof({cname}));')
