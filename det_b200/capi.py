@@ -129,6 +129,7 @@ class FMoeOp(C.Structure):
 
 DET_F32, DET_BF16 = 0, 1
 DET_FF_SWIGLU, DET_FF_REGLU, DET_FF_RELU2 = 0, 1, 2
+DET_MAX_ROUTER = 1024
 DET_DECAY_SIGMOID, DET_DECAY_EXP = 0, 1
 DET_LAYOUT_STREAM = 0x100
 DET_LAYOUT_INT8 = 0x200
