@@ -684,9 +684,23 @@ def hybrid_config(width: int, ff: int, vocab: int, layers: int, window: int = 40
             "layers": [{**kinds[i % 4], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
 
 
+def dopipel_config(width: int, ff: int, vocab: int, runs: int) -> dict:
+    """A Dopipel decoder of `runs` layer runs (6 + 2 for every further pass of its loop) with the layers of a real model: attention
+    and gated recurrences in turn, one layer in three a mixture (64 experts and 8 identity experts, 6 of them per token)."""
+    att = {"type": "attention", "mixer": {"heads": width // 128, "kv_heads": width // 640, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                          "rot": {"base": 10000.0, "dims": 128}}}
+    gru = {"type": "mingru", "mixer": {"width": width}}
+    dense = {"kind": "dense", "ff": ff}
+    inner = ff // 6 // 64 * 64
+    moe = {"kind": "moe", "router": {"experts": 64, "identity": 8, "top": 6}, "expert": {"ff": inner}, "shared": {"ff": inner}}
+    layers = [{**att, "mlp": dense}, {**gru, "mlp": moe}, {**att, "mlp": dense}, {**gru, "mlp": dense}, {**att, "mlp": moe}, {**gru, "mlp": dense}]
+    return {"architecture": "Dopipel", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "canon": {"taps": 4}, "layers": layers,
+            "loop": {"start": 2, "stop": 4, "times": max(1, (runs - 4) // 2)}}
+
+
 def run_hybrid(args, rank: int, world: int, local_rank: int):
-    """The hybrid decoder (bfloat16, seeded random weights) beside the Qwen3.5-shaped quantized model of the same width,
-    feed-forward, vocabulary and depth: prefill, graph-replayed decode of one sequence, and a batched step.  One line; the
+    """The Dopipel decoder and the hybrid decoder (bfloat16, seeded random weights) beside the Qwen3.5-shaped quantized model of the
+    same width, feed-forward, vocabulary and depth: prefill, graph-replayed decode of one sequence, and a batched step.  One line; the
     headline workload is another (`--workload decode`).  Reduced depth: the layers are those of a real model, not their number."""
     import numpy as np
     from det_b200 import capi
@@ -776,14 +790,16 @@ def run_hybrid(args, rank: int, world: int, local_rank: int):
         shape = SHAPES[name]
         cfg = hybrid_config(shape["hidden"], shape["ffn"], shape["vocab"], layers)
         res = {"width": shape["hidden"], "ff": shape["ffn"], "vocab": shape["vocab"], "layers": layers}
-        if "hybrid" in args.arms:
-            m = h.dh_hybrid_new_synth(bk, json.dumps(cfg).encode(), SEED, capi.DET_BF16, ctx, args.chunk)
+        for arm, c in (("hybrid", cfg), ("dopipel", dopipel_config(shape["hidden"], shape["ffn"], shape["vocab"], layers))):
+            if arm not in args.arms.split(","):
+                continue
+            m = h.dh_hybrid_new_synth(bk, json.dumps(c).encode(), SEED, capi.DET_BF16, ctx, args.chunk)
             if not m:
                 raise RuntimeError(h.dh_last_error().decode())
             wb = h.dh_hybrid_weight_bytes(m)
-            res["hybrid"] = {"weight_bytes": wb, **measure(m, shape["vocab"], wb)}
+            res[arm] = {"weight_bytes": wb, **measure(m, shape["vocab"], wb)}
             h.dh_model_free(m)
-        if "qwen35" in args.arms:
+        if "qwen35" in args.arms.split(","):
             m = h.dh_model_new_synth(bk, name.encode(), layers, SEED, ctx, args.chunk)
             if not m:
                 raise RuntimeError(h.dh_last_error().decode())
@@ -795,12 +811,15 @@ def run_hybrid(args, rank: int, world: int, local_rank: int):
     time.sleep(0.3)
     sampler.stop()
     last = sizes[args.sizes.split(",")[-1]]
-    main_arm = last.get("hybrid") or last["qwen35"]
+    arm = next(a for a in ("dopipel", "hybrid", "qwen35") if a in last)
+    main_arm = last[arm]
     print(json.dumps({
-        "metric": "hybrid decoder (Fazilorn) decode tok/s bs1, reduced depth", "value": main_arm["decode"]["value"], "unit": "tok/s",
+        "metric": f"{ {'dopipel': 'Dopipel decoder', 'hybrid': 'hybrid decoder (Fazilorn)', 'qwen35': 'quantized decoder'}[arm]} "
+                  "decode tok/s bs1, reduced depth", "value": main_arm["decode"]["value"], "unit": "tok/s",
         "n_gpus": 1, "steps": K, "warmup": W, "ms_per_step": main_arm["decode"]["ms_per_token"], "higher_is_better": True,
         "scaling": "strong", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": {"layers_built": layers, "pattern": "wkv, gla, latent_attention, gla", "prefill": args.prefill, "chunk": args.chunk,
+        "config": {"layers_built": layers, "pattern": {"hybrid": "wkv, gla, latent_attention, gla", "dopipel": "attention and mingru in turn, a mixture "
+                   "in one layer of three, the middle two layers looped"}, "prefill": args.prefill, "chunk": args.chunk,
                    "l2": "weights streamed per token exceed the 126 MB L2", "hbm_peak_gbs": hbm, "peak_kind": kind,
                    "float_flags": args.float_flags},
         "sizes": sizes, "clocks": sampler.summary(windows)}), flush=True)
@@ -824,9 +843,9 @@ def main():
                          "line says so and is not a result)")
     ap.add_argument("--workload", default="decode", choices=["decode", "serving", "hybrid"],
                     help="decode: the headline batch-1 token loop; serving: many sequences, one batched step per token; "
-                         "hybrid: the bfloat16 hybrid decoder beside the quantized model of equal size")
+                         "hybrid: the bfloat16 decoders (Dopipel, Fazilorn) beside the quantized model of equal size")
     ap.add_argument("--sizes", default="4b,27b", help="hybrid: widths to run, comma separated names of the shapes")
-    ap.add_argument("--arms", default="hybrid,qwen35", help="hybrid: which of the two models to run")
+    ap.add_argument("--arms", default="dopipel,hybrid,qwen35", help="hybrid: which of the models to run")
     ap.add_argument("--float-flags", type=int, default=0, help="hybrid: measurement switches (det_debug_set_float)")
     ap.add_argument("--seqs", type=int, default=32)
     ap.add_argument("--ctx-min", type=int, default=512)

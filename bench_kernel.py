@@ -9,6 +9,10 @@ kernels that a profiler capture needs (a few hundred MB on the device, a handful
     python bench_kernel.py fgemm [N K M]                    # bfloat16 product, default 5120 22528 512 (1 .. 4 rows: the GEMV)
     python bench_kernel.py recur [gla|wkv heads dk dv M]    # linear recurrence, default gla 20 128 256 512
     python bench_kernel.py latent [heads dim rot vdim kv_rank M pos0 window]   # default 40 128 64 128 512 512 1536 4096
+    python bench_kernel.py fattn [heads kv dim vdim M pos0]  # grouped-head attention, default 40 8 128 128 512 1536
+    python bench_kernel.py mingru [n M]                     # minimal gated recurrence, default 5120 512
+    python bench_kernel.py moe [experts identity top ff n M]   # mixture of experts, default 64 8 6 2880 5120 512
+    python bench_kernel.py seam [n M taps]                  # seam between sublayers, default 5120 512 4; taps 0: no convolution
 
 attn: one det_attention call of M tokens behind pos0 cached positions (head_dim 256, random cache contents); tc = 0
 keeps it on the CUDA-core kernels; 2 warm-up calls, then 5 timed ones.
@@ -215,6 +219,95 @@ def latent(argv):
           f"{2 * h * keys * (dim + rot + vdim) / us / 1e6:.1f} TFLOP/s (expanded form); device error word {d.det_last_error()}")
 
 
+def fattn(argv):
+    h, g, dim, vdim, m, pos0 = map(int, argv[1:7]) if len(argv) >= 7 else (40, 8, 128, 128, 512, 1536)
+    d, rng = capi.cuda(), np.random.default_rng(1)
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+    cap, ldy = pos0 + m, h * dim + g * (dim + vdim) + h
+    table = lambda n: _rand(d, rng, (cap, max(1, n // 2)), 0.5)
+    op = capi.FAttnOp(heads=h, kv_heads=g, dim=dim, vdim=vdim, rot_dims=dim, scale=dim ** -0.5, cap=cap, M=m, dtype=capi.DET_BF16,
+                      y=_rand(d, rng, (m, ldy)), ldy=ldy, q_off=0, k_off=h * dim, v_off=(h + g) * dim, gate_off=(h + g) * dim + g * vdim,
+                      rope_cos=table(dim), rope_sin=table(dim), vrope_cos=table(vdim), vrope_sin=table(vdim),
+                      q=d.det_malloc(m * d.det_f_attn_q_ld(h, dim) * 2), out=d.det_malloc(m * h * vdim * 2), ldo=h * vdim, max_pos=cap - 1,
+                      scratch=d.det_malloc(d.det_f_attn_scratch_bytes(vdim)),
+                      seq=capi.SeqRef(one=capi.SeqSlot(cache=_rand(d, rng, (cap, d.det_f_attn_ld(g, dim, vdim)), bf16=True)), pos0=pos0))
+    prep = _time(ev, lambda: d.det_f_attn_prep(C.byref(op), None))
+    us = _time(ev, lambda: d.det_f_attn(C.byref(op), None))
+    pairs = h * sum(pos0 + i + 1 for i in range(m))
+    print(f"det_f_attn heads={h}/{g} dim={dim} vdim={vdim} M={m} pos0={pos0}: prep {prep:.1f} us, attention {us:.1f} us/call, "
+          f"{2 * pairs * (dim + vdim) / us / 1e6:.1f} TFLOP/s, {cap * d.det_f_attn_ld(g, dim, vdim) * 2 / us / 1e3:.0f} GB/s of cache; "
+          f"device error word {d.det_last_error()}")
+
+
+def mingru(argv):
+    n, m = map(int, argv[1:3]) if len(argv) >= 3 else (5120, 512)
+    d, rng = capi.cuda(), np.random.default_rng(1)
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+    copies = max(1, min(16, int(400e6 // (m * n * 12)) + 1))
+    ops = [capi.FMinGruOp(n=n, M=m, dtype=capi.DET_BF16, y=_rand(d, rng, (m, 3 * n)), ldy=3 * n, z_off=0, x_off=n, gate_off=2 * n,
+                          out=d.det_malloc(m * n * 2), ldo=n, seq=capi.SeqRef(one=capi.SeqSlot(s=d.det_malloc(n * 4)))) for _ in range(copies)]
+    turn = [0]
+
+    def call():
+        d.det_f_mingru(C.byref(ops[turn[0] % copies]), None)
+        turn[0] += 1
+    us = _time(ev, call, 4 * copies)
+    print(f"det_f_mingru n={n} M={m}: {us:.1f} us/call, {m * n * 14 / us / 1e3:.0f} GB/s; device error word {d.det_last_error()}")
+
+
+def moe(argv):
+    e, ident, top, ff, n, m = map(int, argv[1:7]) if len(argv) >= 7 else (64, 8, 6, 2880, 5120, 512)
+    d, rng = capi.cuda(), np.random.default_rng(1)
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+
+    def stack(rows, k):
+        lin = _flinear(d, rng, e * rows, k, tiled=False)
+        lin.wt = d.det_malloc(d.det_f_linear_tile_groups_bytes(k, e, rows))
+        d.det_f_linear_tile_groups(C.byref(lin), e, lin.wt, None)
+        return lin
+    up, down, shared = stack(ff, n), stack(n, ff), _flinear(d, rng, n, ff)
+    counts = d.det_malloc((capi.DET_MAX_ROUTER + 1) * 4)
+    d.det_memset(counts, 0, (capi.DET_MAX_ROUTER + 1) * 4, None)
+    zs = [_rand(d, rng, (m, e + ident + 1)) for _ in range(8)]      # other experts every time
+    op = capi.FMoeOp(experts=e, identity=ident, top=top, ff=ff, n=n, M=m, dtype=capi.DET_BF16, ldz=e + ident + 1, x=_rand(d, rng, (m, n), bf16=True),
+                     ldx=n, up=C.pointer(up), down=C.pointer(down), shared=C.pointer(shared), hs=_rand(d, rng, (m, ff), bf16=True), ldhs=ff,
+                     shared_gate=e + ident, out=d.det_malloc(m * n * 4), ldo=n, counts=counts,
+                     scratch=d.det_malloc(d.det_f_moe_scratch_bytes(m, e, top, ff, n, capi.DET_BF16)))
+    turn = [0]
+
+    def call():
+        op.z = zs[turn[0] % 8]
+        d.det_f_moe(C.byref(op), None)
+        turn[0] += 1
+    us = _time(ev, call, 16)
+    real = top * e / (e + ident)
+    print(f"det_f_moe experts={e}+{ident} top={top} ff={ff} n={n} M={m}: {us:.1f} us/call, {4 * m * (real + 0.5) * ff * n / us / 1e6:.0f} TFLOP/s, "
+          f"{(min(e, real * m) * 2 + 1) * ff * n * 2 / us / 1e3:.0f} GB/s of weights (expected experts); device error word {d.det_last_error()}")
+
+
+def seam(argv):
+    n, m, taps = map(int, argv[1:4]) if len(argv) >= 4 else (5120, 512, 4)
+    d, rng = capi.cuda(), np.random.default_rng(1)
+    assert d.det_init() == 0
+    ev = _Events(d.det_cuda_stream())
+    copies = max(1, min(24, int(400e6 // (m * n * 10)) + 1))
+    vec = lambda: _rand(d, rng, n, 0.1)
+    ops = [capi.FSeamOp(x=_rand(d, rng, (m, n)), M=m, n=n, eps=1e-6, y=_rand(d, rng, (m, n)), ldy=n, y_norm=vec(), y_scale=vec(), w=vec(),
+                        conv=_rand(d, rng, (taps, n), 0.1) if taps else None, taps=taps, rstd=d.det_malloc(m * 4), dtype=capi.DET_BF16,
+                        out=d.det_malloc(m * n * 2), ld=n, seq=capi.SeqRef(one=capi.SeqSlot(prev=_rand(d, rng, (max(1, taps), n))))) for _ in range(copies)]
+    turn = [0]
+
+    def call():
+        d.det_f_seam(C.byref(ops[turn[0] % copies]), None)
+        turn[0] += 1
+    us = _time(ev, call, 4 * copies)
+    print(f"det_f_seam n={n} M={m} taps={taps}: {us:.1f} us/call, {m * n * 14 / us / 1e3:.0f} GB/s (x twice, y, output); "
+          f"device error word {d.det_last_error()}")
+
+
 def main(argv):
     kind = argv[0] if argv else "gemv"
     if kind == "umma_peak":
@@ -252,8 +345,9 @@ def main(argv):
         return
     if kind == "attn":
         return attn(argv)
-    if kind in ("fgemm", "recur", "latent"):
-        return {"fgemm": fgemm, "recur": recur, "latent": latent}[kind](argv)
+    cases = {"fgemm": fgemm, "recur": recur, "latent": latent, "fattn": fattn, "mingru": mingru, "moe": moe, "seam": seam}
+    if kind in cases:
+        return cases[kind](argv)
     if kind not in ("gemv", "gemm_tc"):
         raise SystemExit(__doc__)
     n, k, bits, m = (17408, 5120, 6, 1 if kind == "gemv" else 512)

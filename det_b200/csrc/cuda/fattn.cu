@@ -1,7 +1,8 @@
 // Attention over grouped key/value heads (include/det_b200.h, det_fattn_op): rotated queries and keys, optionally rotated
 // values whose sum is turned back by the query's position, one output gate per head.
 //
-//   k_fattn_prep    rotation; queries into a row of their own, keys and values into the sequence's cache.
+//   k_fattn_prep    rotation; queries into a row of their own, keys and values into the sequence's cache.  One row per sequence
+//                   in bfloat16 needs no such launch: k_fattn_dec rotates the row itself.
 //   k_fattn_flash   a run of tokens, bfloat16: the flash loop of flash.cuh, 64 query rows of a head.
 //   k_fattn_dec     few rows, bfloat16: the query heads of one key/value head are the 16 rows of an MMA tile, a CTA's four
 //                   warps and further CTAs split the keys.  Bound by the bytes of the cache.
@@ -138,6 +139,42 @@ __device__ __forceinline__ bool last_to_arrive(unsigned* counter, int splits) {
     if (last) __threadfence();
     return last;
 }
+// A CTA adds the pieces of `nh` heads of a row from h0 on.  fac: room for nh * (splits + 1) floats.
+template <class T>
+__device__ __forceinline__ void merge_block(const AttnArgs& a, int row, int pos, int h0, int nh, float* fac) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, pr = 2 + a.vd, S = a.splits;
+    const float* first = a.part + ((size_t)row * a.heads + h0) * S * pr;
+    for (int r = warp; r < nh; r += warps) {
+        const float* p = first + (size_t)r * S * pr;
+        float m = -INFINITY, l = 0.0f;
+        for (int s = lane; s < S; s += 32) m = fmaxf(m, __ldcg(p + (size_t)s * pr));
+        m = warp_max(m);
+        for (int s = lane; s < S; s += 32) {
+            const float2 ml = __ldcg(reinterpret_cast<const float2*>(p + (size_t)s * pr));
+            const float f = exp2f(ml.x - m);
+            fac[r * (S + 1) + s] = f;
+            l = fmaf(f, ml.y, l);
+        }
+        l = warp_sum(l);
+        if (lane == 0) fac[r * (S + 1) + S] = 1.0f / l;
+    }
+    __syncthreads();
+    const int vp = a.vd / 2;
+    for (int i = threadIdx.x; i < nh * vp; i += blockDim.x) {
+        const int r = i / vp, v = (i - r * vp) * 2;
+        if (v >= a.vdim) continue;
+        const float* p = first + (size_t)r * S * pr + 2 + v;
+        const float* f = fac + r * (S + 1);
+        float o0 = 0.0f, o1 = 0.0f;
+#pragma unroll 16
+        for (int s = 0; s < S; s++) {
+            const float2 x = __ldcg(reinterpret_cast<const float2*>(p + (size_t)s * pr));
+            o0 = fmaf(f[s], x.x, o0);
+            o1 = fmaf(f[s], x.y, o1);
+        }
+        put_out<T>(a, row, pos, h0 + r, v, o0 * f[S], o1 * f[S]);
+    }
+}
 // A warp adds the pieces of one row and head.
 template <class T>
 __device__ __forceinline__ void merge_pieces(const AttnArgs& a, int row, int pos, int h) {
@@ -162,17 +199,18 @@ __device__ __forceinline__ void merge_pieces(const AttnArgs& a, int row, int pos
 }
 
 // ------------------------------------------------------------------------------------------------------ few rows
-constexpr int AD_WARPS = 4, AD_KEYS = 16, AD_STAGES = 3, AD_HEADS = 16;
+constexpr int AD_WARPS = 4, AD_KEYS = 16, AD_STAGES = 3, AD_HEADS = 16, AT_TARGET = 2 * 148;   // AT_TARGET: CTAs of a split launch
 
 static size_t dec_smem(int kd, int dv) {
     const int ldk = ((kd + 15) & ~15) + 8;
     const size_t ring = ((size_t)AD_HEADS * ldk + (size_t)AD_WARPS * AD_STAGES * AD_KEYS * (ldk + dv + 8)) * 2;
-    return std::max(ring, (size_t)AD_WARPS * AD_HEADS * (dv + 2) * sizeof(float));
+    return std::max({ring, (size_t)AD_WARPS * AD_HEADS * (dv + 2) * sizeof(float), (size_t)AD_HEADS * (AT_TARGET + 1) * sizeof(float)});
 }
 
-// grid (splits, kv_heads * head blocks, rows); DV = value dimensions rounded up to a multiple of 64.
+// grid (splits, kv_heads * head blocks, rows); DV = value dimensions rounded up to a multiple of 64.  `fused`: q has not been
+// rotated nor k and v been cached yet (every row is its sequence's only one).
 template <int DV>
-__global__ void __launch_bounds__(AD_WARPS * 32) k_fattn_dec(const AttnArgs a) {
+__global__ void __launch_bounds__(AD_WARPS * 32) k_fattn_dec(const AttnArgs a, int fused) {
     extern __shared__ __align__(16) uint8_t asm_[];
     const int dqp = (a.kd + 15) & ~15, ldk = dqp + 8;
     constexpr int LDV = DV + 8;
@@ -183,21 +221,42 @@ __global__ void __launch_bounds__(AD_WARPS * 32) k_fattn_dec(const AttnArgs a) {
     const int hblocks = (a.per_kv + AD_HEADS - 1) / AD_HEADS, g = blockIdx.y / hblocks, hb = blockIdx.y % hblocks;
     const int h0 = g * a.per_kv + hb * AD_HEADS, nh = min(AD_HEADS, a.per_kv - hb * AD_HEADS), row = blockIdx.z;
     pdl_trigger();
-    {
-        const int words = (AD_HEADS * ldk + AD_WARPS * AD_STAGES * AD_KEYS * (ldk + LDV)) / 8;      // pads stay zero
-        for (int i = threadIdx.x; i < words; i += AD_WARPS * 32) reinterpret_cast<uint4*>(asm_)[i] = make_uint4(0, 0, 0, 0);
-    }
+    // what the copies leave unwritten enters products: all of it, or the rows of queries that do not exist
+    const bool pads = dqp != a.kd || DV != a.vd;
+    const int words = (AD_HEADS * ldk + (pads ? AD_WARPS * AD_STAGES * AD_KEYS * (ldk + LDV) : 0)) / 8;
+    for (int i = threadIdx.x; i < words; i += AD_WARPS * 32) reinterpret_cast<uint4*>(asm_)[i] = make_uint4(0, 0, 0, 0);
+    __syncthreads();
     pdl_wait();
     const int pos = position_of(a.seq, row);
     const int lo = blockIdx.x * a.per_split, hi = min(pos + 1, lo + a.per_split);
-    __syncthreads();
-    const bf16* q = static_cast<const bf16*>(a.q) + (size_t)row * a.ldq + (size_t)h0 * a.kd;
-    for (int i = threadIdx.x; i < nh * (a.kd / 8); i += AD_WARPS * 32) {
-        const int h = i / (a.kd / 8), v = i % (a.kd / 8);
-        *reinterpret_cast<uint4*>(Q + h * ldk + v * 8) = *reinterpret_cast<const uint4*>(q + h * a.kd + v * 8);
+    bf16* cache = static_cast<bf16*>(slot_of(a.seq, row).cache);
+    if (fused) {
+        const float* y = a.y + (size_t)row * a.ldy;
+        const int kp = a.kd / 2, vp = a.vd / 2;
+        bf16* c = cache + (size_t)pos * a.ld;
+        const int own = hi == pos + 1 && lo < hi ? kp + vp : 0;               // the CTAs that read the new key also cache it
+        for (int i = threadIdx.x; i < nh * kp + own; i += AD_WARPS * 32) {
+            if (i < nh * kp) {
+                const int h = i / kp, e = (i - h * kp) * 2;
+                float2 v = rotated_pair(y + a.q_off + (h0 + h) * a.dim, e, a.dim, a.rot_dims, a.rope_cos, a.rope_sin, pos);
+                put_pair(Q + h * ldk + e, make_float2(v.x * a.scale, v.y * a.scale));
+            } else if (i < nh * kp + kp) {
+                const int e = (i - nh * kp) * 2;
+                put_pair(c + g * a.kd + e, rotated_pair(y + a.k_off + g * a.dim, e, a.dim, a.rot_dims, a.rope_cos, a.rope_sin, pos));
+            } else {
+                const int e = (i - nh * kp - kp) * 2;
+                put_pair(c + a.kv_heads * a.kd + g * a.vd + e,
+                         rotated_pair(y + a.v_off + g * a.vdim, e, a.vdim, a.vrope_cos ? a.vdim : 0, a.vrope_cos, a.vrope_sin, pos));
+            }
+        }
+    } else {
+        const bf16* q = static_cast<const bf16*>(a.q) + (size_t)row * a.ldq + (size_t)h0 * a.kd;
+        for (int i = threadIdx.x; i < nh * (a.kd / 8); i += AD_WARPS * 32) {
+            const int h = i / (a.kd / 8), v = i % (a.kd / 8);
+            *reinterpret_cast<uint4*>(Q + h * ldk + v * 8) = *reinterpret_cast<const uint4*>(q + h * a.kd + v * 8);
+        }
     }
     __syncthreads();
-    const bf16* cache = static_cast<const bf16*>(slot_of(a.seq, row).cache);
     const int kvec = a.kd / 8, tvec = kvec + a.vd / 8;
     auto fetch = [&](int k0, int stage) {
         if (k0 < hi)
@@ -299,7 +358,7 @@ __global__ void __launch_bounds__(AD_WARPS * 32) k_fattn_dec(const AttnArgs a) {
         }
     }
     if (a.splits == 1 || !last_to_arrive(a.counters + (size_t)row * gridDim.y + blockIdx.y, a.splits)) return;
-    for (int r = warp; r < nh; r += AD_WARPS) merge_pieces<bf16>(a, row, pos, h0 + r);
+    merge_block<bf16>(a, row, pos, h0, nh, reinterpret_cast<float*>(asm_));
 }
 
 // ------------------------------------------------------------------------------------------------------ 32-bit, any size
@@ -393,7 +452,6 @@ __global__ void __launch_bounds__(AS_WARPS * 32) k_fattn_simt(const AttnArgs a) 
 }
 
 // ------------------------------------------------------------------------------------------------------ host side
-constexpr int AT_TARGET = 2 * 148;      // CTAs of a split launch
 static bool takes_flash(const det_fattn_op& op, const AttnArgs& a) {
     const int dv = (a.vd + 63) / 64 * 64;
     return op.dtype == DET_BF16 && !op.seq.table && !op.seq.pos && op.M >= 32 && !(float_flags() & 8) && a.vd <= 256 &&
@@ -402,12 +460,15 @@ static bool takes_flash(const det_fattn_op& op, const AttnArgs& a) {
 static bool takes_dec(const det_fattn_op& op, const AttnArgs& a) {
     return op.dtype == DET_BF16 && !(float_flags() & 8) && a.vd <= 256 && dec_smem(a.kd, (a.vd + 63) / 64 * 64) <= 220 * 1024;
 }
+// Calls whose rows k_fattn_dec rotates and caches itself: one row per sequence.
+static bool rotates_itself(const det_fattn_op& op, const AttnArgs& a) {
+    return (op.seq.table || op.M == 1) && takes_dec(op, a) && !takes_flash(op, a);
+}
 // Key ranges per row: enough CTAs to fill the device, at least 64 keys each.
-static void plan(AttnArgs& a, int blocks, int max_pos) {
+static void plan(AttnArgs& a, int blocks, int max_pos, int target) {
     const long long ctas = (long long)a.M * blocks;
     const int keys = max_pos + 1;
-    int s = (int)std::min<long long>((keys + 63) / 64, AT_TARGET / ctas);
-    a.counters = nullptr;
+    int s = (int)std::min<long long>((keys + 63) / 64, target / ctas);
     int n = 0;
     unsigned* counters = fsplit_counters(&n);
     if (ctas > n) s = 1;
@@ -427,7 +488,7 @@ static void launch_flash(const AttnArgs& a, cudaStream_t q) {
     launch_plain(k_fattn_flash<DV>, dim3((a.M + FL_ROWS - 1) / FL_ROWS, a.heads), dim3(FL_WARPS * 32), smem, q, a);
 }
 template <int DV>
-static void launch_dec(AttnArgs a, int max_pos, cudaStream_t q) {
+static void launch_dec(AttnArgs a, int max_pos, bool fused, cudaStream_t q) {
     const size_t smem = dec_smem(a.kd, DV);
     static size_t configured = 0;
     if (smem > configured) {
@@ -435,13 +496,13 @@ static void launch_dec(AttnArgs a, int max_pos, cudaStream_t q) {
         configured = smem;
     }
     const int blocks = a.kv_heads * ((a.per_kv + AD_HEADS - 1) / AD_HEADS);
-    plan(a, blocks, max_pos);
-    launch_pdl(k_fattn_dec<DV>, dim3(a.splits, blocks, a.M), dim3(AD_WARPS * 32), smem, q, 1, a);
+    plan(a, blocks, max_pos, AT_TARGET / 2);
+    launch_pdl(k_fattn_dec<DV>, dim3(a.splits, blocks, a.M), dim3(AD_WARPS * 32), smem, q, 1, a, fused ? 1 : 0);
 }
 template <class T>
 static void launch_simt(AttnArgs a, int max_pos, cudaStream_t q) {
     const int blocks = (a.heads + AS_WARPS - 1) / AS_WARPS, np = (std::max(a.kd, a.vd) + 63) / 64;
-    plan(a, blocks, max_pos);
+    plan(a, blocks, max_pos, AT_TARGET);
     const dim3 grid(a.splits, blocks, a.M), block(AS_WARPS * 32);
     if (np <= 2) launch_pdl(k_fattn_simt<T, 2>, grid, block, 0, q, 1, a);
     else if (np <= 4) launch_pdl(k_fattn_simt<T, 4>, grid, block, 0, q, 1, a);
@@ -484,7 +545,7 @@ size_t det_f_attn_scratch_bytes(int vdim) { return (size_t)AT_TARGET * AD_HEADS 
 
 void det_f_attn_prep(const det_fattn_op* op, cudaStream_t st) {
     const AttnArgs a = attn_args(op);
-    if (op->M <= 0) return;
+    if (op->M <= 0 || rotates_itself(*op, a)) return;
     const int pairs = (a.heads + a.kv_heads) * a.kd / 2 + a.kv_heads * a.vd / 2;
     const int pieces = std::max(1, std::min((pairs + PREP_THREADS - 1) / PREP_THREADS, 4 * sm_count() / op->M));
     if (op->dtype == DET_BF16) launch_pdl(k_fattn_prep<bf16>, dim3(op->M, pieces), dim3(PREP_THREADS), 0, queue_of(st), 1, a);
@@ -503,10 +564,11 @@ void det_f_attn(const det_fattn_op* op, cudaStream_t st) {
         else if (dv == 3) launch_flash<192>(a, q);
         else launch_flash<256>(a, q);
     } else if (takes_dec(*op, a)) {
-        if (dv == 1) launch_dec<64>(a, op->max_pos, q);
-        else if (dv == 2) launch_dec<128>(a, op->max_pos, q);
-        else if (dv == 3) launch_dec<192>(a, op->max_pos, q);
-        else launch_dec<256>(a, op->max_pos, q);
+        const bool fused = rotates_itself(*op, a);
+        if (dv == 1) launch_dec<64>(a, op->max_pos, fused, q);
+        else if (dv == 2) launch_dec<128>(a, op->max_pos, fused, q);
+        else if (dv == 3) launch_dec<192>(a, op->max_pos, fused, q);
+        else launch_dec<256>(a, op->max_pos, fused, q);
     } else if (op->dtype == DET_BF16) {
         launch_simt<bf16>(a, op->max_pos, q);
     } else {

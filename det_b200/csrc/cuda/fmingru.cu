@@ -4,7 +4,7 @@
 //   k_fmingru_step   one token per row (decode, batches): elementwise.
 //   k_fmingru_scan   a run of tokens: a CTA takes 32 channels, its warps consecutive pieces of SCAN_T tokens.  A warp reduces its
 //                    piece to (product of 1 - z, state from zero), the pieces' entry states follow from those in order, and
-//                    the warp replays its piece from registers: one read of the inputs, 32 * SCAN_T tokens per round.
+//                    the warp replays its piece from registers: one read of the inputs, SCAN_WARPS * SCAN_T tokens per round.
 // Bound by the bytes of the fp32 rows.
 #include "fops.cuh"
 #include <algorithm>
@@ -27,7 +27,7 @@ __global__ void __launch_bounds__(256) k_fmingru_step(const det_fmingru_op a) {
     put(static_cast<T*>(a.out) + (size_t)row * a.ldo + i, v * silu_fast(y[a.gate_off + i]));
 }
 
-constexpr int SCAN_T = 8, SCAN_WARPS = 32;
+constexpr int SCAN_T = 8, SCAN_WARPS = 16;      // 512 threads: three CTAs an SM
 
 template <class T>
 __global__ void __launch_bounds__(SCAN_WARPS * 32) k_fmingru_scan(const det_fmingru_op a) {

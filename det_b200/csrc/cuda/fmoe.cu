@@ -130,12 +130,24 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32) k_fmoe_route(const MoeArgs a
 // ------------------------------------------------------------------------------------------------------ few rows
 constexpr int MD_WARPS = 16, MD_THREADS = MD_WARPS * 32, MD_ROWS = 4, MD_MAX = 64;   // MD_MAX: second halves of a row
 
+__device__ __forceinline__ void load_eight(const float* p, float (&v)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void load_eight(const bf16* p, float (&v)[8]) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    v[0] = bf_lo(a.x); v[1] = bf_hi(a.x); v[2] = bf_lo(a.y); v[3] = bf_hi(a.y);
+    v[4] = bf_lo(a.z); v[5] = bf_hi(a.z); v[6] = bf_lo(a.w); v[7] = bf_hi(a.w);
+}
+
 // grid (CTAs, rows).  xs: the row's weighted first halves side by side, each padded to a multiple of 8, two planes of four.
 template <class T>
 __global__ void __launch_bounds__(MD_THREADS, 1) k_fmoe_down(const MoeArgs a, int wsplit) {
     extern __shared__ __align__(16) float xs[];
     __shared__ const bf16* base[MD_MAX];
-    __shared__ int ld[MD_MAX], start[MD_MAX + 1];
+    __shared__ int ld[MD_MAX], start[MD_MAX + 1], from[MD_MAX];
+    __shared__ float scale[MD_MAX];
     __shared__ float red[2][MD_WARPS][MD_ROWS];
     __shared__ int count;
     pdl_trigger();
@@ -144,71 +156,82 @@ __global__ void __launch_bounds__(MD_THREADS, 1) k_fmoe_down(const MoeArgs a, in
     const int* sel = a.sel + (size_t)row * a.top;
     const float* extra = a.extra + row * 2;
     const int fp = (a.ff + 7) & ~7, sp = (a.sk + 7) & ~7;
-    if (threadIdx.x == 0) {
+    // the segments of the row's product: its chosen experts in order, then the shared one
+    if (warp == 0) {
         int c = 0;
-        for (int k = 0; k < a.top; k++)
-            if (sel[k] < a.experts) {
-                base[c] = a.down + (size_t)sel[k] * a.n * a.ldd;
-                ld[c] = a.ldd;
-                start[c] = c * fp;
-                c++;
+        for (int k0 = 0; k0 < a.top; k0 += 32) {
+            const int k = k0 + lane, e = k < a.top ? sel[k] : a.experts;
+            const unsigned real = __ballot_sync(FULL, e < a.experts);
+            if (e < a.experts) {
+                const int i = c + __popc(real & ((1u << lane) - 1u));
+                base[i] = a.down + (size_t)e * a.n * a.ldd;
+                ld[i] = a.ldd;
+                start[i] = i * fp;
+                from[i] = k;
+                scale[i] = a.weight[(size_t)row * a.top + k];
             }
-        start[c] = c * fp;
-        if (a.sdown) {
-            base[c] = a.sdown;
-            ld[c] = a.lds;
-            c++;
-            start[c] = start[c - 1] + sp;
+            c += __popc(real);
         }
-        count = c;
+        if (lane == 0) {
+            start[c] = c * fp;
+            if (a.sdown) {
+                base[c] = a.sdown;
+                ld[c] = a.lds;
+                from[c] = -1;
+                scale[c] = extra[1];
+                c++;
+                start[c] = start[c - 1] + sp;
+            }
+            count = c;
+        }
     }
     __syncthreads();
     const int nseg = count, kt = start[nseg], half = kt / 2;
-    int at = 0;
-    for (int k = 0; k < a.top; k++) {
-        if (sel[k] >= a.experts) continue;
-        const T* h = static_cast<const T*>(a.h1) + ((size_t)row * a.top + k) * a.ldh;
-        const float w = a.weight[(size_t)row * a.top + k];
-        for (int i = threadIdx.x; i < fp; i += MD_THREADS) {
-            const int j = at + i;
-            xs[((j >> 2) & 1) * half + (j >> 3) * 4 + (j & 3)] = i < a.ff ? to_f(h[i]) * w : 0.0f;
-        }
-        at += fp;
-    }
-    if (a.sdown) {
-        const T* h = static_cast<const T*>(a.hs) + (size_t)row * a.ldhs;
-        for (int i = threadIdx.x; i < sp; i += MD_THREADS) {
-            const int j = at + i;
-            xs[((j >> 2) & 1) * half + (j >> 3) * 4 + (j & 3)] = i < a.sk ? to_f(h[i]) * extra[1] : 0.0f;
-        }
-    }
-    __syncthreads();
-    const float identity = extra[0];
     const int group = warp / wsplit, part = warp % wsplit, qpc = MD_WARPS / wsplit;
     const int nquads = (a.n + MD_ROWS - 1) / MD_ROWS, stride = qpc * gridDim.x, kstep = wsplit * 256;
-    int quad = blockIdx.x * qpc + group, buf = 0;
+    int quad = blockIdx.x * qpc + group, buf = 0, seg = 0;
+    const int k_first = (part * 32 + lane) * 8;
+    auto load = [&](int qd, int k, uint4 (&w)[MD_ROWS]) {
+        if (k >= kt || qd >= nquads) {
+#pragma unroll
+            for (int r = 0; r < MD_ROWS; r++) w[r] = make_uint4(0, 0, 0, 0);
+            return;
+        }
+        while (k >= start[seg + 1]) seg++;
+        const bf16* p = base[seg] + (k - start[seg]);
+        const size_t l = ld[seg];
+#pragma unroll
+        for (int r = 0; r < MD_ROWS; r++) w[r] = __ldcs(reinterpret_cast<const uint4*>(p + min(qd * MD_ROWS + r, a.n - 1) * l));
+    };
+    uint4 w0[MD_ROWS], w1[MD_ROWS];
+    load(quad, k_first, w0);
+    {
+        int s = 0;
+        for (int j = threadIdx.x * 8; j < kt; j += MD_THREADS * 8) {
+            while (j >= start[s + 1]) s++;
+            const int i = j - start[s], n = (from[s] < 0 ? a.sk : a.ff) - i;
+            const T* h = from[s] < 0 ? static_cast<const T*>(a.hs) + (size_t)row * a.ldhs : static_cast<const T*>(a.h1) + ((size_t)row * a.top + from[s]) * a.ldh;
+            float v[8];
+            load_eight(h + i, v);
+#pragma unroll
+            for (int t = 0; t < 8; t++) v[t] = t < n ? v[t] * scale[s] : 0.0f;
+            *reinterpret_cast<float4*>(xs + (j >> 1)) = make_float4(v[0], v[1], v[2], v[3]);
+            *reinterpret_cast<float4*>(xs + half + (j >> 1)) = make_float4(v[4], v[5], v[6], v[7]);
+        }
+    }
+    const float identity = extra[0];
+    __syncthreads();
     for (int b = blockIdx.x * qpc; b < nquads; b += stride, quad += stride, buf ^= 1) {
         const bool live = quad < nquads;
         if (live) {
             float acc[MD_ROWS] = {0.0f, 0.0f, 0.0f, 0.0f};
-            int seg = 0;
-            auto load = [&](int k, uint4 (&w)[MD_ROWS]) {
-                if (k >= kt) {
-#pragma unroll
-                    for (int r = 0; r < MD_ROWS; r++) w[r] = make_uint4(0, 0, 0, 0);
-                    return;
-                }
-                while (k >= start[seg + 1]) seg++;
-                const bf16* p = base[seg] + (k - start[seg]);
-                const size_t l = ld[seg];
-#pragma unroll
-                for (int r = 0; r < MD_ROWS; r++) w[r] = __ldcs(reinterpret_cast<const uint4*>(p + min(quad * MD_ROWS + r, a.n - 1) * l));
-            };
-            uint4 w0[MD_ROWS], w1[MD_ROWS];
-            const int k_first = (part * 32 + lane) * 8;
-            load(k_first, w0);
             for (int k = k_first; k < kt; k += kstep) {
-                load(k + kstep, w1);
+                if (k + kstep < kt) {
+                    load(quad, k + kstep, w1);
+                } else {                              // the next quad's first weights, ahead of this one's sums
+                    seg = 0;
+                    load(quad + stride, k_first, w1);
+                }
                 const float4 xa = *reinterpret_cast<const float4*>(xs + (k >> 1)), xb = *reinterpret_cast<const float4*>(xs + half + (k >> 1));
 #pragma unroll
                 for (int r = 0; r < MD_ROWS; r++) {
@@ -305,26 +328,58 @@ __global__ void __launch_bounds__(MG_WARPS * 32) k_fmoe_gather(const MoeArgs a) 
     for (int i = a.ff + lane; i < a.ldh; i += 32) put(h + i, 0.0f);
 }
 
-// out holds the shared expert's second half when there is one
-template <class T>
+// out holds the shared expert's second half when there is one.  V columns per thread and pass.
+template <class T, int V>
 __global__ void __launch_bounds__(256) k_fmoe_combine(const MoeArgs a) {
+    __shared__ int rows[DET_MAX_ROUTER];
+    __shared__ float weights[DET_MAX_ROUTER];
     pdl_trigger();
     pdl_wait();
     const int row = blockIdx.x;
     if (row == 0 && blockIdx.y == 0)
         for (int e = threadIdx.x; e < a.experts; e += 256) a.counts[e] = 0;     // for the next call
-    const int* place = a.rank + (size_t)row * a.top;
-    const float* weight = a.weight + (size_t)row * a.top;
+    for (int k = threadIdx.x; k < a.top; k += 256) {
+        const int p = a.rank[(size_t)row * a.top + k];
+        rows[k] = max(p, 0);
+        weights[k] = p >= 0 ? a.weight[(size_t)row * a.top + k] : 0.0f;
+    }
     const float identity = a.extra[row * 2], gate = a.extra[row * 2 + 1];
     const T* x = static_cast<const T*>(a.x) + (size_t)row * a.ldx;
     float* out = a.out + (size_t)row * a.ldo;
-    for (int i = blockIdx.y * 256 + threadIdx.x; i < a.n; i += gridDim.y * 256) {
-        float v = a.sdown ? gate * out[i] : 0.0f;
-        if (identity != 0.0f) v = fmaf(identity, to_f(x[i]), v);
-        for (int k = 0; k < a.top; k++)
-            if (place[k] >= 0) v = fmaf(weight[k], a.yp[(size_t)place[k] * a.n + i], v);
-        out[i] = v;
+    __syncthreads();
+    for (int i = (blockIdx.y * 256 + threadIdx.x) * V; i < a.n; i += gridDim.y * 256 * V) {
+        float v[V];
+#pragma unroll
+        for (int j = 0; j < V; j++) v[j] = a.sdown ? gate * out[i + j] : 0.0f;
+        if (identity != 0.0f)
+#pragma unroll
+            for (int j = 0; j < V; j++) v[j] = fmaf(identity, to_f(x[i + j]), v[j]);
+#pragma unroll 4
+        for (int k = 0; k < a.top; k++) {
+            if (weights[k] == 0.0f) continue;                                  // x itself: no row of its own
+            const float* y = a.yp + (size_t)rows[k] * a.n + i;
+            if constexpr (V == 4) {
+                const float4 f = *reinterpret_cast<const float4*>(y);
+                v[0] = fmaf(weights[k], f.x, v[0]);
+                v[1] = fmaf(weights[k], f.y, v[1]);
+                v[2] = fmaf(weights[k], f.z, v[2]);
+                v[3] = fmaf(weights[k], f.w, v[3]);
+            } else {
+                v[0] = fmaf(weights[k], *y, v[0]);
+            }
+        }
+        if constexpr (V == 4) *reinterpret_cast<float4*>(out + i) = make_float4(v[0], v[1], v[2], v[3]);
+        else out[i] = v[0];
     }
+}
+
+template <class T>
+static void launch_combine(const MoeArgs& a, cudaStream_t q) {
+    const bool wide = a.n % 4 == 0 && a.ldo % 4 == 0 && (reinterpret_cast<uintptr_t>(a.out) & 15) == 0;
+    const int cols = 256 * (wide ? 4 : 1);
+    const dim3 grid(a.M, std::max(1, std::min((a.n + cols - 1) / cols, 8 * sm_count() / a.M)));
+    if (wide) launch_pdl(k_fmoe_combine<T, 4>, grid, dim3(256), 0, q, 1, a);
+    else launch_pdl(k_fmoe_combine<T, 1>, grid, dim3(256), 0, q, 1, a);
 }
 
 // ------------------------------------------------------------------------------------------------------ host side
@@ -434,6 +489,7 @@ void det_f_moe(const det_fmoe_op* op, cudaStream_t st) {
 
     const dim3 rgrid((a.M + ROUTE_WARPS - 1) / ROUTE_WARPS), rblock(ROUTE_WARPS * 32);
     if (outputs <= 64) launch_pdl(k_fmoe_route<2>, rgrid, rblock, 0, q, 1, a, few ? 0 : 1);
+    else if (outputs <= 128) launch_pdl(k_fmoe_route<4>, rgrid, rblock, 0, q, 1, a, few ? 0 : 1);
     else if (outputs <= 256) launch_pdl(k_fmoe_route<8>, rgrid, rblock, 0, q, 1, a, few ? 0 : 1);
     else launch_pdl(k_fmoe_route<32>, rgrid, rblock, 0, q, 1, a, few ? 0 : 1);
     if (few) {
@@ -479,9 +535,8 @@ void det_f_moe(const det_fmoe_op* op, cudaStream_t st) {
         g.ldy = op->ldo;
         det_f_gemm(&g, st);
     }
-    const dim3 cgrid(a.M, std::max(1, std::min((a.n + 255) / 256, 4 * sm_count() / a.M)));
-    if (bf) launch_pdl(k_fmoe_combine<bf16>, cgrid, dim3(256), 0, q, 1, a);
-    else launch_pdl(k_fmoe_combine<float>, cgrid, dim3(256), 0, q, 1, a);
+    if (bf) launch_combine<bf16>(a, q);
+    else launch_combine<float>(a, q);
 }
 
 }  // extern "C"

@@ -53,8 +53,10 @@ __device__ __forceinline__ float row_sum(float v, float* sh, float* slots, int c
     return s;
 }
 
-// `own`: every row of the call has its own history (or the call is one row).
-template <class T, int V>
+// `own`: every row of the call has its own history (or the call is one row).  ONE: a thread has one vector of the row, which
+// stays in registers, and loads what does not depend on the kernel before ahead of the wait; otherwise the row goes through
+// shared memory, which leaves room for eight CTAs an SM.
+template <class T, int V, bool ONE>
 __global__ void __launch_bounds__(SEAM_THREADS) k_fseam(const det_fseam_op a, int cs, int own) {
     extern __shared__ __align__(16) float buf[];        // this CTA's columns
     __shared__ float sh[32];
@@ -62,41 +64,69 @@ __global__ void __launch_bounds__(SEAM_THREADS) k_fseam(const det_fseam_op a, in
     pdl_trigger();
     const int row = blockIdx.x / cs, piece = blockIdx.x % cs;
     const int per = ((a.n + V - 1) / V + cs - 1) / cs * V, c0 = min(a.n, piece * per), c1 = min(a.n, c0 + per);
+    const int first = c0 + (int)threadIdx.x * V;
     float* x = a.x + (size_t)row * a.n;
+    auto each = [&](auto f) {
+        if constexpr (ONE) {
+            if (first < c1) f(first);
+        } else {
+            for (int i = first; i < c1; i += SEAM_THREADS * V) f(i);
+        }
+    };
+    Vec<V> mine, xv, yn, ys, w;
+    auto keep = [&](int i, const Vec<V>& v) {
+        if constexpr (ONE) mine = v;
+        else store_vec(buf + (i - c0), v);
+    };
+    auto kept = [&](int i) {
+        if constexpr (ONE) return mine;
+        else return load_vec<V>(buf + (i - c0));
+    };
+    if constexpr (ONE)
+        each([&](int i) {
+            if (a.y) yn = load_vec<V>(a.y_norm + i);
+            if (a.y && a.y_scale) ys = load_vec<V>(a.y_scale + i);
+            if (a.w) w = load_vec<V>(a.w + i);
+        });
     if (cs > 1) cooperative_groups::this_cluster().sync();      // peers run before anything is pushed to them
     pdl_wait();
+    if constexpr (ONE) each([&](int i) { xv = load_vec<V>(x + i); });
     float ss = 0.0f;
     if (a.y) {
         const float* y = a.y + (size_t)row * a.ldy;
-        for (int i = c0 + threadIdx.x * V; i < c1; i += SEAM_THREADS * V) {
+        each([&](int i) {
             const Vec<V> v = load_vec<V>(y + i);
 #pragma unroll
             for (int j = 0; j < V; j++) ss = fmaf(v.v[j], v.v[j], ss);
-            store_vec(buf + (i - c0), v);
-        }
+            keep(i, v);
+        });
         const float rs = 1.0f / sqrtf(row_sum(ss, sh, slots[0], cs) / (float)a.n + a.eps);
         ss = 0.0f;
-        for (int i = c0 + threadIdx.x * V; i < c1; i += SEAM_THREADS * V) {
-            const Vec<V> v = load_vec<V>(buf + (i - c0)), w = load_vec<V>(a.y_norm + i);
-            Vec<V> r = load_vec<V>(x + i), s;
-            if (a.y_scale) s = load_vec<V>(a.y_scale + i);
+        each([&](int i) {
+            const Vec<V> v = kept(i);
+            if constexpr (!ONE) {
+                xv = load_vec<V>(x + i);
+                yn = load_vec<V>(a.y_norm + i);
+                if (a.y_scale) ys = load_vec<V>(a.y_scale + i);
+            }
+            Vec<V> r = xv;
 #pragma unroll
             for (int j = 0; j < V; j++) {
-                float t = v.v[j] * rs * w.v[j];
-                if (a.y_scale) t *= s.v[j];
+                float t = v.v[j] * rs * yn.v[j];
+                if (a.y_scale) t *= ys.v[j];
                 r.v[j] += t;
                 ss = fmaf(r.v[j], r.v[j], ss);
             }
             store_vec(x + i, r);
-            store_vec(buf + (i - c0), r);
-        }
+            keep(i, r);
+        });
     } else {
-        for (int i = c0 + threadIdx.x * V; i < c1; i += SEAM_THREADS * V) {
-            const Vec<V> v = load_vec<V>(x + i);
+        each([&](int i) {
+            const Vec<V> v = ONE ? xv : load_vec<V>(x + i);
 #pragma unroll
             for (int j = 0; j < V; j++) ss = fmaf(v.v[j], v.v[j], ss);
-            store_vec(buf + (i - c0), v);
-        }
+            keep(i, v);
+        });
     }
     if (!a.out) return;
     float rs = 1.0f;
@@ -107,15 +137,16 @@ __global__ void __launch_bounds__(SEAM_THREADS) k_fseam(const det_fseam_op a, in
     }
     T* out = static_cast<T*>(a.out) + (size_t)row * a.ld;
     float* prev = a.conv ? slot_of(a.seq, row).prev : nullptr;
-    for (int i = c0 + threadIdx.x * V; i < c1; i += SEAM_THREADS * V) {
-        Vec<V> h = load_vec<V>(buf + (i - c0));
+    each([&](int i) {
+        Vec<V> h = kept(i);
         if (a.w) {
-            const Vec<V> w = load_vec<V>(a.w + i);
+            if constexpr (!ONE) w = load_vec<V>(a.w + i);
 #pragma unroll
             for (int j = 0; j < V; j++) h.v[j] = h.v[j] * rs * w.v[j];
         }
         if (a.conv) {
             Vec<V> o = h;
+#pragma unroll 4
             for (int t = 0; t < a.taps - 1; t++) {
                 const Vec<V> p = load_vec<V>(prev + (size_t)t * a.n + i), c = load_vec<V>(a.conv + (size_t)t * a.n + i);
 #pragma unroll
@@ -129,7 +160,7 @@ __global__ void __launch_bounds__(SEAM_THREADS) k_fseam(const det_fseam_op a, in
             h = o;
         }
         store_vec(out + i, h);
-    }
+    });
 }
 
 // ---------------------------------------------------------------------------------------------- runs of tokens
@@ -190,19 +221,27 @@ __global__ void __launch_bounds__(SEAM_THREADS) k_fconv(const det_fseam_op a) {
     }
 }
 
+template <class T, int V, bool ONE>
+static void launch_row(const det_fseam_op& op, int cs, int own, cudaStream_t q) {
+    size_t smem = 0;
+    if constexpr (!ONE) {
+        smem = (size_t)(((op.n + V - 1) / V + cs - 1) / cs * V) * sizeof(float);
+        static size_t configured = 48 * 1024;
+        if (smem > configured) {
+            DETB_CUDA_OK(cudaFuncSetAttribute(k_fseam<T, V, ONE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            configured = smem;
+        }
+    }
+    launch_pdl(k_fseam<T, V, ONE>, dim3(op.M * cs), dim3(SEAM_THREADS), smem, q, cs, op, cs, own);
+}
 template <class T, int V>
 static void launch_seam(const det_fseam_op& op, cudaStream_t q) {
     const bool own = op.seq.table != nullptr || op.M == 1 || !op.conv;
+    auto vecs = [&](int cs) { return ((op.n + V - 1) / V + cs - 1) / cs; };      // of a CTA
     int cs = 1;
-    while (cs < SEAM_MAX_CLUSTER && (long long)op.M * cs * 2 <= sm_count() && op.n > cs * SEAM_THREADS * V) cs *= 2;
-    const int per = ((op.n + V - 1) / V + cs - 1) / cs * V;
-    const size_t smem = (size_t)per * sizeof(float);
-    static size_t configured = 48 * 1024;
-    if (smem > configured) {
-        DETB_CUDA_OK(cudaFuncSetAttribute(k_fseam<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        configured = smem;
-    }
-    launch_pdl(k_fseam<T, V>, dim3(op.M * cs), dim3(SEAM_THREADS), smem, q, cs, op, cs, own ? 1 : 0);
+    while (cs < SEAM_MAX_CLUSTER && vecs(cs) > SEAM_THREADS && (long long)op.M * cs * 2 <= sm_count()) cs *= 2;
+    if (vecs(cs) <= SEAM_THREADS) launch_row<T, V, true>(op, cs, own ? 1 : 0, q);
+    else launch_row<T, V, false>(op, cs, own ? 1 : 0, q);
     if (own || !op.out) return;
     if (op.taps <= 4) {
         launch_pdl(k_fconv<T, V, 4>, dim3((op.M + CONV_ROWS - 1) / CONV_ROWS, (op.n + SEAM_THREADS * V - 1) / (SEAM_THREADS * V)),
@@ -223,10 +262,11 @@ extern "C" void det_f_seam(const det_fseam_op* op, cudaStream_t st) {
     DETB_REQUIRE(!op->conv || (op->w && op->taps >= 1 && op->taps <= DET_MAX_TAPS), "seam: bad convolution");
     if (op->M <= 0) return;
     DETB_REQUIRE(!op->conv || op->seq.table || op->M == 1 || op->rstd, "seam: a run of tokens needs scratch");
+    DETB_REQUIRE((size_t)op->n * sizeof(float) <= smem_optin() - 4096, "seam: the row is too long");
     auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    // four columns at a time where every row allows it
     const bool wide = op->n % 4 == 0 && op->ldy % 4 == 0 && aligned(op->x) && aligned(op->y) && aligned(op->y_norm) && aligned(op->y_scale) &&
                       aligned(op->w) && aligned(op->conv) && aligned(op->out) && (op->seq.table || aligned(op->seq.one.prev));
-    DETB_REQUIRE((size_t)op->n * sizeof(float) <= smem_optin() - 4096, "seam: the row is too long");
     cudaStream_t q = queue_of(st);
     if (op->dtype == DET_BF16) {
         if (wide) launch_seam<bf16, 4>(*op, q);

@@ -586,8 +586,8 @@ void det_f_seam(const det_fseam_op* op, cudaStream_t st);
  * a head's output is turned back by the query's position.  A cache row holds the rotated keys and values of one position in
  * the activation type (det_f_attn_ld elements: every head's key and value padded to a multiple of 8).
  * det_f_attn_prep writes the rows' cache entries and the scaled rotated queries q (activation type, det_f_attn_q_ld elements
- * a row); det_f_attn: softmax(scale * q . k) over the positions j <= i, out[row][head * vdim + j] = value * sigmoid(gate).
- * max_pos bounds the positions; the caller guarantees cap > max_pos.                                                   */
+ * a row), unless det_f_attn will do so itself for this call.  det_f_attn: softmax(scale * q . k) over the positions j <= i,
+ * out[row][head * vdim + j] = value * sigmoid(gate).  max_pos bounds the positions; the caller guarantees cap > max_pos. */
 typedef struct {
     int heads, kv_heads, dim, vdim, rot_dims;
     float scale;
